@@ -41,6 +41,8 @@ SHARPI_API int sharpi_embed_gather(const int* ids, const void* table, int table_
 //   rows == nullptr:  x[t] += delta[t] (written back); out[t] = x[t] * rsqrt(mean(x[t]^2)+eps) * w
 //                     (w == nullptr: the weightless norm, src/SharpInference.Cpu/SimdKernels.cs:4252-4283)
 //   rows != nullptr:  r = rows[t]; v = x[r] + delta[r] (x untouched); out[t] = norm(v)
+//   w2 / out2:        (sharpi_add_rmsnorm_pair) the same normalised row under a second weight, for blocks whose two
+//                     sublayers read the same stream through norms of their own; `out32` is then the second's copy
 // `out` has dtype out_dtype; `out32` (optional) receives the same values in fp32, for
 // consumers that must not see them rounded (the expert router).
 // One block of NORM_THREADS threads per row whatever the batch, so the order of the
@@ -59,10 +61,11 @@ constexpr int NORM_CACHE_FLOATS = 12288;     // 48 KB
 // added their own elements and the block's tree were that of 32 warps), so that a row gives the same bits
 // whichever of the two kernels a step of its size takes: this thread stands for the virtual threads
 // t, t + 256, t + 512, t + 768.
-template <typename TO, bool CACHED, bool WIDE_ORDER>
+template <typename TO, bool CACHED, bool WIDE_ORDER, bool PAIR = false>
 __global__ void __launch_bounds__(NORM_THREADS)
 add_rmsnorm_kernel(float* x, const float* __restrict__ delta, const float* __restrict__ w, float eps,
-                   const int* __restrict__ rows, int H, TO* __restrict__ out, float* __restrict__ out32) {
+                   const int* __restrict__ rows, int H, TO* __restrict__ out, float* __restrict__ out32,
+                   const float* __restrict__ w2, TO* __restrict__ out2) {
     __shared__ float scratch[32];
     extern __shared__ float row_s[];
     pdl_wait();
@@ -127,8 +130,12 @@ add_rmsnorm_kernel(float* x, const float* __restrict__ delta, const float* __res
         for (int k = 0; k < NORM_UNROLL; ++k) {
             const int i = i0 + k * NORM_THREADS;
             if (i < H) {
-                const float y = v[k] * scale * ww[k];
+                float y = v[k] * scale * ww[k];
                 orow[i] = from_float<TO>(y);
+                if (PAIR) {
+                    y = v[k] * scale * w2[i];
+                    out2[(size_t)t * H + i] = from_float<TO>(y);
+                }
                 if (o32) o32[i] = y;
             }
         }
@@ -143,17 +150,19 @@ add_rmsnorm_kernel(float* x, const float* __restrict__ delta, const float* __res
 constexpr int NORM_WIDE_THREADS = 1024;
 constexpr int NORM_WIDE_ROWS = 128;       // steps of up to this many rows take it
 
-template <typename TO>
+template <typename TO, bool PAIR = false>
 __global__ void __launch_bounds__(NORM_WIDE_THREADS)
 add_rmsnorm_wide_kernel(float* x, const float* __restrict__ delta, const float* __restrict__ w, float eps,
-                        const int* __restrict__ rows, int H, TO* __restrict__ out, float* __restrict__ out32) {
+                        const int* __restrict__ rows, int H, TO* __restrict__ out, float* __restrict__ out32,
+                        const float* __restrict__ w2, TO* __restrict__ out2) {
     __shared__ float scratch[32];
     // the weight is written by no kernel: it may be on its way before the kernel ahead has finished
-    float ww[NORM_UNROLL];
+    float ww[NORM_UNROLL], ww2[PAIR ? NORM_UNROLL : 1];
 #pragma unroll
     for (int k = 0; k < NORM_UNROLL; ++k) {
         const int i = threadIdx.x + k * NORM_WIDE_THREADS;
         ww[k] = (i < H) ? (w ? w[i] : 1.0f) : 0.0f;
+        if (PAIR) ww2[k] = (i < H) ? w2[i] : 0.0f;
     }
     pdl_wait();
     const int t = blockIdx.x;
@@ -186,34 +195,38 @@ add_rmsnorm_wide_kernel(float* x, const float* __restrict__ delta, const float* 
     for (int k = 0; k < NORM_UNROLL; ++k) {
         const int i = threadIdx.x + k * NORM_WIDE_THREADS;
         if (i < H) {
-            const float y = v[k] * scale * ww[k];
+            float y = v[k] * scale * ww[k];
             orow[i] = from_float<TO>(y);
+            if (PAIR) {
+                y = v[k] * scale * ww2[k];
+                out2[(size_t)t * H + i] = from_float<TO>(y);
+            }
             if (o32) o32[i] = y;
         }
     }
 }
 
-template <typename TO>
+template <typename TO, bool PAIR = false>
 static int launch_norm(float* x, const float* delta, const float* w, float eps, const int* rows, int T, int H, TO* out,
-                       float* out32, cudaStream_t stream) {
+                       float* out32, cudaStream_t stream, const float* w2 = nullptr, TO* out2 = nullptr) {
     if (H <= NORM_WIDE_THREADS * NORM_UNROLL) {
         // few rows: latency counts (2.9 against 3.8 us at one row of 5120); many rows: bandwidth (33 against 49 us at
         // 2048 rows); the two kernels add in the same order, so the choice does not show in the result
         if (T <= NORM_WIDE_ROWS) {
-            auto kern = add_rmsnorm_wide_kernel<TO>;
-            SHARPI_LAUNCH_PDL(kern, T, NORM_WIDE_THREADS, 0, stream, x, delta, w, eps, rows, H, out, out32);
+            auto kern = add_rmsnorm_wide_kernel<TO, PAIR>;
+            SHARPI_LAUNCH_PDL(kern, T, NORM_WIDE_THREADS, 0, stream, x, delta, w, eps, rows, H, out, out32, w2, out2);
         } else {
-            auto kern = add_rmsnorm_kernel<TO, true, true>;
-            SHARPI_LAUNCH_PDL(kern, T, NORM_THREADS, (size_t)H * sizeof(float), stream, x, delta, w, eps, rows, H, out, out32);
+            auto kern = add_rmsnorm_kernel<TO, true, true, PAIR>;
+            SHARPI_LAUNCH_PDL(kern, T, NORM_THREADS, (size_t)H * sizeof(float), stream, x, delta, w, eps, rows, H, out, out32, w2, out2);
         }
         return SHARPI_OK;
     }
     if (H <= NORM_CACHE_FLOATS) {
-        auto kern = add_rmsnorm_kernel<TO, true, false>;
-        SHARPI_LAUNCH_PDL(kern, T, NORM_THREADS, (size_t)H * sizeof(float), stream, x, delta, w, eps, rows, H, out, out32);
+        auto kern = add_rmsnorm_kernel<TO, true, false, PAIR>;
+        SHARPI_LAUNCH_PDL(kern, T, NORM_THREADS, (size_t)H * sizeof(float), stream, x, delta, w, eps, rows, H, out, out32, w2, out2);
     } else {
-        auto kern = add_rmsnorm_kernel<TO, false, false>;
-        SHARPI_LAUNCH_PDL(kern, T, NORM_THREADS, 0, stream, x, delta, w, eps, rows, H, out, out32);
+        auto kern = add_rmsnorm_kernel<TO, false, false, PAIR>;
+        SHARPI_LAUNCH_PDL(kern, T, NORM_THREADS, 0, stream, x, delta, w, eps, rows, H, out, out32, w2, out2);
     }
     return SHARPI_OK;
 }
@@ -224,6 +237,17 @@ SHARPI_API int sharpi_add_rmsnorm(float* x, const float* delta, const float* w, 
     if (H <= 0) return SHARPI_BAD_ARGUMENT;
     if (out_dtype == SHARPI_F32) return launch_norm<float>(x, delta, w, eps, rows, T, H, (float*)out, out32, stream);
     if (out_dtype == SHARPI_BF16) return launch_norm<bf16>(x, delta, w, eps, rows, T, H, (bf16*)out, out32, stream);
+    return SHARPI_BAD_ARGUMENT;
+}
+
+SHARPI_API int sharpi_add_rmsnorm_pair(float* x, const float* delta, const float* w1, const float* w2, float eps, int T,
+                                       int H, void* out1, void* out2, int out_dtype, float* out32, cudaStream_t stream) {
+    if (T <= 0) return SHARPI_OK;
+    if (H <= 0 || !w1 || !w2) return SHARPI_BAD_ARGUMENT;
+    if (out_dtype == SHARPI_F32)
+        return launch_norm<float, true>(x, delta, w1, eps, nullptr, T, H, (float*)out1, out32, stream, w2, (float*)out2);
+    if (out_dtype == SHARPI_BF16)
+        return launch_norm<bf16, true>(x, delta, w1, eps, nullptr, T, H, (bf16*)out1, out32, stream, w2, (bf16*)out2);
     return SHARPI_BAD_ARGUMENT;
 }
 
@@ -629,5 +653,143 @@ SHARPI_API int sharpi_sigmoid_gate(const void* o, const float* g, void* out, int
         SHARPI_LAUNCH_PDL(sigmoid_gate_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)o, g, (bf16*)out, n, cols, g_ld);
     else
         return SHARPI_BAD_ARGUMENT;
+    return SHARPI_OK;
+}
+
+// ---------------------------------------------------------------------------------------
+// The gated activation of a feed-forward with biases, written into a column range:
+//   g = gate_up[m, i] + bias[i],  u = gate_up[m, I + i] + bias[I + i]        (bias nullable)
+//   limit == 0:  out[m, i] = act(g) * u                                     (relu^2, tanh-GELU or SiLU)
+//   limit > 0:   g = min(g, limit), u = clamp(u, -limit, limit), out[m, i] = g sigmoid(1.702 g) (u + 1)
+// `out` rows are `ld` elements apart; behind the I elements `ones` columns of 1 and `zeros` columns of 0 are written (the
+// product that reads the range can carry its bias as weight columns there, and a width its kernels like).
+// ---------------------------------------------------------------------------------------
+__device__ __forceinline__ float clamped_gate(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+template <typename TO, int ACT, bool CLAMP>
+__global__ void __launch_bounds__(256)
+gated_cols_kernel(const float* gate_up, const float* __restrict__ bias, TO* out, int I, int ld, int ones, int tail, float limit) {
+    pdl_wait();
+    const size_t m = blockIdx.x;
+    const int i = blockIdx.y * blockDim.x + threadIdx.x;
+    if (i >= I + tail) return;
+    float y;
+    if (i < I) {
+        const float g = gate_up[m * 2 * I + i] + (bias ? bias[i] : 0.0f);
+        const float u = gate_up[m * 2 * I + I + i] + (bias ? bias[I + i] : 0.0f);
+        y = CLAMP ? clamped_gate(g, u, limit) : activate<ACT>(g) * u;
+    } else {
+        y = i < I + ones ? 1.0f : 0.0f;
+    }
+    out[m * ld + i] = from_float<TO>(y);
+}
+
+// four elements a thread (16-byte loads), sizes and places that are multiples of four
+template <typename TO, int ACT, bool CLAMP>
+__global__ void __launch_bounds__(256)
+gated_cols_vec4_kernel(const float* gate_up, const float* __restrict__ bias, TO* out, int I, int ld, int ones, int tail, float limit) {
+    pdl_wait();
+    const size_t m = blockIdx.x;
+    const int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+    if (i >= I + tail) return;
+    float y[4];
+    if (i < I) {
+        float4 g = *reinterpret_cast<const float4*>(gate_up + m * 2 * I + i);
+        float4 u = *reinterpret_cast<const float4*>(gate_up + m * 2 * I + I + i);
+        if (bias) {
+            const float4 bg = *reinterpret_cast<const float4*>(bias + i), bu = *reinterpret_cast<const float4*>(bias + I + i);
+            g.x += bg.x; g.y += bg.y; g.z += bg.z; g.w += bg.w;
+            u.x += bu.x; u.y += bu.y; u.z += bu.z; u.w += bu.w;
+        }
+        const float gs[4] = {g.x, g.y, g.z, g.w}, us[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = CLAMP ? clamped_gate(gs[j], us[j], limit) : activate<ACT>(gs[j]) * us[j];
+    } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = i + j < I + ones ? 1.0f : 0.0f;
+    }
+    TO* dst = out + m * ld + i;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) dst[j] = from_float<TO>(y[j]);
+}
+
+template <typename TO, int ACT, bool CLAMP>
+static int launch_gated_cols(const float* gate_up, const float* bias, TO* out, int M, int I, int ld, int ones, int tail,
+                             float limit, cudaStream_t stream) {
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(bias);
+    if (I % 4 == 0 && tail % 4 == 0 && (ptrs & 15) == 0) {
+        auto kern = gated_cols_vec4_kernel<TO, ACT, CLAMP>;
+        SHARPI_LAUNCH_PDL(kern, dim3(M, ((I + tail) / 4 + 255) / 256), 256, 0, stream, gate_up, bias, out, I, ld, ones, tail, limit);
+    } else {
+        auto kern = gated_cols_kernel<TO, ACT, CLAMP>;
+        SHARPI_LAUNCH_PDL(kern, dim3(M, (I + tail + 255) / 256), 256, 0, stream, gate_up, bias, out, I, ld, ones, tail, limit);
+    }
+    return SHARPI_OK;
+}
+
+SHARPI_API int sharpi_gated_cols(const float* gate_up, const float* bias, void* out, int out_dtype, int M, int I, int ld,
+                                 int ones, int zeros, int act, float limit, cudaStream_t stream) {
+    if (M <= 0 || I <= 0) return SHARPI_OK;
+    const int tail = ones + zeros;
+    if (ones < 0 || zeros < 0 || ld < I + tail || (I + tail + 255) / 256 > 65535 || !(limit >= 0.0f)) return SHARPI_BAD_ARGUMENT;
+#define COLS_CASE(TO)                                                                                                       \
+    do {                                                                                                                    \
+        TO* o = (TO*)out;                                                                                                   \
+        if (limit > 0.0f) return launch_gated_cols<TO, ACT_SILU, true>(gate_up, bias, o, M, I, ld, ones, tail, limit, stream); \
+        if (act == ACT_RELU2) return launch_gated_cols<TO, ACT_RELU2, false>(gate_up, bias, o, M, I, ld, ones, tail, 0.0f, stream); \
+        if (act == ACT_GELU_TANH) return launch_gated_cols<TO, ACT_GELU_TANH, false>(gate_up, bias, o, M, I, ld, ones, tail, 0.0f, stream); \
+        if (act == ACT_SILU) return launch_gated_cols<TO, ACT_SILU, false>(gate_up, bias, o, M, I, ld, ones, tail, 0.0f, stream); \
+        return SHARPI_BAD_ARGUMENT;                                                                                         \
+    } while (0)
+    if (out_dtype == SHARPI_F32) COLS_CASE(float);
+    if (out_dtype == SHARPI_BF16) COLS_CASE(bf16);
+#undef COLS_CASE
+    return SHARPI_BAD_ARGUMENT;
+}
+
+// out[t, h dv + i] = o[t, h, i] * sigmoid(g[t, h]) * scale for i < dv: a gate of one number per head on attention outputs
+// whose heads are D >= dv elements apart, laid side by side in a column range of a wider matrix.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+gate_heads_kernel(const TO* o, const float* g, int ld_g, TO* out, int ld_out, int heads, int D, int dv, float scale) {
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < heads * dv; i += gridDim.y * blockDim.x) {
+        const int h = i / dv, e = i - h * dv;
+        const float f = scale / (1.0f + expf(-g[t * ld_g + h]));
+        out[t * ld_out + i] = from_float<TO>(to_float(o[(t * heads + h) * D + e]) * f);
+    }
+}
+
+SHARPI_API int sharpi_gate_heads(const void* o, const float* g, int ld_g, void* out, int ld_out, int dtype, int T, int heads,
+                                 int D, int dv, float scale, cudaStream_t stream) {
+    if (T <= 0) return SHARPI_OK;
+    if (heads <= 0 || dv <= 0 || D < dv || ld_g < heads || ld_out < heads * dv) return SHARPI_BAD_ARGUMENT;
+    int by = (heads * dv + 1023) / 1024;
+    const dim3 grid(T, by > 64 ? 64 : by);
+    if (dtype == SHARPI_F32)
+        SHARPI_LAUNCH_PDL(gate_heads_kernel<float>, grid, 256, 0, stream, (const float*)o, g, ld_g, (float*)out, ld_out, heads, D, dv, scale);
+    else if (dtype == SHARPI_BF16)
+        SHARPI_LAUNCH_PDL(gate_heads_kernel<bf16>, grid, 256, 0, stream, (const bf16*)o, g, ld_g, (bf16*)out, ld_out, heads, D, dv, scale);
+    else
+        return SHARPI_BAD_ARGUMENT;
+    return SHARPI_OK;
+}
+
+// y = cap * tanh(y / cap), in place (float32): a cap on the logits
+__global__ void softcap_kernel(float* y, float cap, long long n) {
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) y[i] = cap * tanhf(y[i] / cap);
+}
+
+SHARPI_API int sharpi_softcap(float* y, float cap, long long n, cudaStream_t stream) {
+    if (n <= 0) return SHARPI_OK;
+    if (!(cap > 0.0f)) return SHARPI_BAD_ARGUMENT;
+    SHARPI_LAUNCH_PDL(softcap_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, y, cap, n);
     return SHARPI_OK;
 }

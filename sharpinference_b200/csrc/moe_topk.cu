@@ -7,8 +7,15 @@
 //                 (softmax over the chosen): the k experts with the largest logits z are chosen and their weights are
 //                 scale * exp(z_i - max) / sum over the chosen of exp(z_j - max): the other experts' logits do not
 //                 enter.
+//                 `scoring` = 2 (softmax over all): s = softmax(z) over every expert; the choice score is s + correction;
+//                 with `n_groups` > 1 the experts form equal groups of neighbours, a group's score is its largest choice
+//                 score, and only experts of the `keep` best groups may be chosen (the lowest index among equal groups).
+//                 Weights as for the sigmoid (scale * s / (sum + 1e-20) when `renormalize`).
+//                 `gate_w` [H] (optional): one more row, gate_out[t] = sigmoid(gate_w . h_t), the gate of a shared expert.
 //   pair_tokens   after the (row, choice) pairs have been sorted by expert: the row each sorted pair belongs to.
 //   combine       out[t] = add[t] + sum over the row's k pairs of y[pair], in the order of the choices.
+//   combine_full  out[t] = add[t] + gate[t] shared[t] + sum over the row's k pairs of (y[pair], or weight[pair] h[t] for a
+//                 choice beyond the experts that have weights: an identity expert), in the order of the choices.
 //
 // The reference routes on the host, one row at a time (src/SharpInference.Engine/ForwardPass.cs:2021-2098); here
 // routing stays on the device so that a step's rows can be sorted by expert for grouped products.
@@ -26,8 +33,9 @@ __global__ void __launch_bounds__(TOPK_WARPS * 32)
 router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                    int T, int H, int E, int k, float scale, int renormalize, int* __restrict__ expert_id,
                    float* __restrict__ weight, float* __restrict__ scores_out, int stage_rows,
-                   const float* __restrict__ bias, int scoring) {
-    extern __shared__ float smem[];                       // per row s [E], choice [E]; then the rows [ROWS][H] if they fit
+                   const float* __restrict__ bias, int scoring, int n_groups, int keep, const float* __restrict__ gate_w,
+                   float* __restrict__ gate_out) {
+    extern __shared__ float smem[];                       // per row s [E], choice [E]; group scores; then the rows [ROWS][H] if they fit
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * TOPK_ROWS;
     const int rows = min(TOPK_ROWS, T - t0);
@@ -35,14 +43,14 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
 #pragma unroll
     for (int r = 0; r < TOPK_ROWS; ++r) row[r] = h + (size_t)(t0 + min(r, rows - 1)) * H;
     if (stage_rows) {                                     // the rows are read from memory once, by all warps together
-        float* rows_s = smem + (size_t)TOPK_ROWS * 2 * E;
+        float* rows_s = smem + (size_t)TOPK_ROWS * (2 * E + n_groups);
         for (int i = threadIdx.x; i < rows * H; i += TOPK_WARPS * 32) rows_s[i] = h[(size_t)t0 * H + i];
         __syncthreads();
 #pragma unroll
         for (int r = 0; r < TOPK_ROWS; ++r) row[r] = rows_s + (size_t)min(r, rows - 1) * H;
     }
-    for (int e = warp; e < E; e += TOPK_WARPS) {
-        const float* w = wr + (size_t)e * H;
+    for (int e = warp; e < E + (gate_w ? 1 : 0); e += TOPK_WARPS) {
+        const float* w = e < E ? wr + (size_t)e * H : gate_w;
         float acc[TOPK_ROWS][4];
 #pragma unroll
         for (int r = 0; r < TOPK_ROWS; ++r)
@@ -68,12 +76,13 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
         }
 #pragma unroll
         for (int r = 0; r < TOPK_ROWS; ++r) {
-            const float z = warp_sum((acc[r][0] + acc[r][1]) + (acc[r][2] + acc[r][3])) + (bias ? bias[e] : 0.0f);
-            if (lane == 0 && r < rows) {
-                const float s = scoring == 1 ? z : 1.0f / (1.0f + expf(-z));
+            const float z = warp_sum((acc[r][0] + acc[r][1]) + (acc[r][2] + acc[r][3])) + (bias && e < E ? bias[e] : 0.0f);
+            if (lane == 0 && r < rows && e == E) gate_out[t0 + r] = 1.0f / (1.0f + expf(-z));
+            if (lane == 0 && r < rows && e < E) {
+                const float s = scoring >= 1 ? z : 1.0f / (1.0f + expf(-z));
                 smem[(size_t)r * 2 * E + e] = s;
                 smem[(size_t)r * 2 * E + E + e] = correction ? s + correction[e] : s;
-                if (scores_out) scores_out[(size_t)(t0 + r) * E + e] = s;
+                if (scores_out && scoring != 2) scores_out[(size_t)(t0 + r) * E + e] = s;
             }
         }
     }
@@ -82,6 +91,42 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
     const int t = t0 + warp;
     float* s_s = smem + (size_t)warp * 2 * E;
     float* c_s = s_s + E;
+    if (scoring == 2) {
+        float m = -INFINITY, sum = 0.0f;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, s_s[e]);
+        m = warp_max(m);
+        for (int e = lane; e < E; e += 32) {
+            const float x = expf(s_s[e] - m);
+            s_s[e] = x;
+            sum += x;
+        }
+        sum = warp_sum(sum);
+        for (int e = lane; e < E; e += 32) {
+            const float s = s_s[e] / sum;
+            s_s[e] = s;
+            c_s[e] = correction ? s + correction[e] : s;
+            if (scores_out) scores_out[(size_t)t * E + e] = s;
+        }
+        __syncwarp();
+        if (n_groups > 1 && keep < n_groups) {
+            float* g_s = smem + (size_t)TOPK_ROWS * 2 * E + (size_t)warp * n_groups;       // a group's largest choice score
+            const int per = E / n_groups;
+            for (int g = lane; g < n_groups; g += 32) {
+                float best = -INFINITY;
+                for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, c_s[e]);
+                g_s[g] = best;
+            }
+            __syncwarp();
+            // a group stays when fewer than `keep` groups are ahead of it (larger score, or equal and lower index)
+            for (int g = lane; g < n_groups; g += 32) {
+                int ahead = 0;
+                for (int o = 0; o < n_groups; ++o) ahead += g_s[o] > g_s[g] || (g_s[o] == g_s[g] && o < g);
+                if (ahead >= keep)
+                    for (int e = g * per; e < (g + 1) * per; ++e) c_s[e] = -INFINITY;
+            }
+            __syncwarp();
+        }
+    }
     float total = 0.0f, top = 0.0f;
     int mine = 0;                                          // lane j keeps the j-th choice
     for (int j = 0; j < k; ++j) {
@@ -115,28 +160,51 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
         if (lane < k) weight[(size_t)t * k + lane] = expf(s_s[mine] - top) * (scale / total);
         return;
     }
-    const float factor = renormalize ? scale / total : scale;
+    const float factor = renormalize ? scale / (scoring == 2 ? total + 1e-20f : total) : scale;
     if (lane < k) weight[(size_t)t * k + lane] = s_s[mine] * factor;      // k <= 32 is checked by the host
 }
 
-SHARPI_API int sharpi_router_topk(const float* h, const float* wr, const float* correction, int T, int H, int E, int k,
-                                  float scale, int renormalize, int* expert_id, float* weight, float* scores_out,
-                                  const float* bias, int scoring, cudaStream_t stream) {
+static int router_topk_impl(const float* h, const float* wr, const float* correction, int T, int H, int E, int k,
+                            float scale, int renormalize, int* expert_id, float* weight, float* scores_out,
+                            const float* bias, int scoring, int n_groups, int keep, const float* gate_w, float* gate_out,
+                            cudaStream_t stream) {
     if (T <= 0) return SHARPI_OK;
-    if (H <= 0 || E <= 0 || k <= 0 || k > E || k > 32 || (scoring != 0 && scoring != 1)) return SHARPI_BAD_ARGUMENT;
+    if (H <= 0 || E <= 0 || k <= 0 || k > E || k > 32) return SHARPI_BAD_ARGUMENT;
     const int per_cta = T > TOPK_MANY_ROWS ? 4 : 1;
-    size_t smem = (size_t)per_cta * 2 * E * sizeof(float);
+    size_t smem = (size_t)per_cta * (2 * E + n_groups) * sizeof(float);
     if (smem > 48 * 1024) return SHARPI_BAD_ARGUMENT;
     const int stage_rows = smem + (size_t)per_cta * H * sizeof(float) <= 48 * 1024;
     if (stage_rows) smem += (size_t)per_cta * H * sizeof(float);
     if (per_cta == 4)
         router_topk_kernel<4><<<(T + 3) / 4, TOPK_WARPS * 32, smem, stream>>>(
-            h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring);
+            h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring,
+            n_groups, keep, gate_w, gate_out);
     else
         router_topk_kernel<1><<<T, TOPK_WARPS * 32, smem, stream>>>(
-            h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring);
+            h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring,
+            n_groups, keep, gate_w, gate_out);
     SHARPI_CHECK_LAUNCH();
     return SHARPI_OK;
+}
+
+SHARPI_API int sharpi_router_topk(const float* h, const float* wr, const float* correction, int T, int H, int E, int k,
+                                  float scale, int renormalize, int* expert_id, float* weight, float* scores_out,
+                                  const float* bias, int scoring, cudaStream_t stream) {
+    if (scoring != 0 && scoring != 1) return SHARPI_BAD_ARGUMENT;
+    return router_topk_impl(h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, bias, scoring,
+                            0, 0, nullptr, nullptr, stream);
+}
+
+// The softmax over all experts, with groups (n_groups >= 1, keep of them; k must fit the kept groups' experts) and the gate row
+SHARPI_API int sharpi_router_groups(const float* h, const float* wr, const float* correction, int T, int H, int E, int k,
+                                    float scale, int renormalize, int n_groups, int keep, const float* gate_w,
+                                    float* gate_out, int* expert_id, float* weight, float* scores_out,
+                                    cudaStream_t stream) {
+    if (n_groups < 1 || E % n_groups != 0 || keep < 1 || keep > n_groups || k > keep * (E / n_groups) ||
+        (gate_w == nullptr) != (gate_out == nullptr))
+        return SHARPI_BAD_ARGUMENT;
+    return router_topk_impl(h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, nullptr, 2,
+                            n_groups, keep, gate_w, gate_out, stream);
 }
 
 __global__ void pair_tokens_kernel(const int* __restrict__ sorted_pairs, int P, int k, int* __restrict__ tokens) {
@@ -190,5 +258,67 @@ SHARPI_API int sharpi_moe_combine(const float* y, const float* add, float* out, 
     if (by > 64) by = 64;
     moe_combine_kernel<<<dim3(T, by), 256, 0, stream>>>(y, add, out, k, H);
     SHARPI_CHECK_LAUNCH();
+    return SHARPI_OK;
+}
+
+template <int VEC>
+__global__ void __launch_bounds__(256)
+moe_combine_full_kernel(const float* y, const int* expert, const float* weight, const float* h, const float* shared,
+                        const float* gate, const float* add, float* out, int E, int k, int H) {
+    pdl_wait();
+    const int t = blockIdx.x;
+    const float gt = shared ? (gate ? gate[t] : 1.0f) : 0.0f;
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; i < H; i += gridDim.y * blockDim.x * VEC) {
+        float acc[VEC];
+        const size_t at = (size_t)t * H + i;
+        auto read = [&](const float* p, float* v) {
+            if (VEC == 4) {
+                const float4 x = *reinterpret_cast<const float4*>(p);
+                v[0] = x.x; v[1 % VEC] = x.y; v[2 % VEC] = x.z; v[3 % VEC] = x.w;
+            } else {
+                v[0] = *p;
+            }
+        };
+        float v[VEC], x[VEC];
+        read(h + at, x);
+#pragma unroll
+        for (int u = 0; u < VEC; ++u) acc[u] = 0.0f;
+        if (add) read(add + at, acc);
+        if (shared) {
+            read(shared + at, v);
+#pragma unroll
+            for (int u = 0; u < VEC; ++u) acc[u] = fmaf(gt, v[u], acc[u]);
+        }
+        for (int j = 0; j < k; ++j) {
+            const size_t pair = (size_t)t * k + j;
+            if (expert[pair] < E) {
+                read(y + pair * H + i, v);
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) acc[u] += v[u];
+            } else {
+                const float w = weight[pair];
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) acc[u] = fmaf(w, x[u], acc[u]);
+            }
+        }
+        if (VEC == 4) *reinterpret_cast<float4*>(out + at) = make_float4(acc[0], acc[1 % VEC], acc[2 % VEC], acc[3 % VEC]);
+        else out[at] = acc[0];
+    }
+}
+
+// `shared`, `gate` and `add` may be null; `out` may be `add`.  Choices >= E are identity experts.
+SHARPI_API int sharpi_moe_combine_full(const float* y, const int* expert, const float* weight, const float* h,
+                                       const float* shared, const float* gate, const float* add, float* out, int T, int E,
+                                       int k, int H, cudaStream_t stream) {
+    if (T <= 0 || H <= 0) return SHARPI_OK;
+    if (k <= 0 || E < 0) return SHARPI_BAD_ARGUMENT;
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared) |
+                           reinterpret_cast<uintptr_t>(add) | reinterpret_cast<uintptr_t>(out);
+    const bool vec = H % 4 == 0 && (ptrs & 15) == 0;
+    int by = (H / (vec ? 4 : 1) + 255) / 256;
+    if (by > 64) by = 64;
+    if (by < 1) by = 1;
+    if (vec) SHARPI_LAUNCH_PDL(moe_combine_full_kernel<4>, dim3(T, by), 256, 0, stream, y, expert, weight, h, shared, gate, add, out, E, k, H);
+    else SHARPI_LAUNCH_PDL(moe_combine_full_kernel<1>, dim3(T, by), 256, 0, stream, y, expert, weight, h, shared, gate, add, out, E, k, H);
     return SHARPI_OK;
 }

@@ -622,3 +622,175 @@ SHARPI_API int sharpi_qkv_post_wide(const float* qkv, int ld, const int* positio
                                  has_kv, stream);
     return SHARPI_BAD_ARGUMENT;
 }
+
+// ---------------------------------------------------------------------------------------------------------
+// The same pass for layers whose projected channels first go through a short causal convolution over time, each
+// channel by itself and without an activation:
+//
+//     y_t[c] = sum_j w[j][c] u_(t - (taps - 1) + j)[c]      (the last tap is the current token's, zeros before the start)
+//
+// over q (nq * dk), k (nkv * dk) and v (nkv * dv), which lie side by side in `proj` from column `col0`; then the rotation of
+// the first `rot` elements of q and k, the store of q and the scatter of k and v into the pages, heads padded with
+// zeros to D.  Inputs before a portion's first row come from the request's state (its last taps - 1 projected values,
+// oldest first).  One warp serves one head of one row; the warp of a portion's FIRST row also serves the head's next
+// taps - 2 rows, which are the only other ones that read the state, and then moves the state on to the portion's last
+// inputs: so nobody reads what it overwrites.  float32 throughout; a row's numbers depend on its own inputs alone.
+// ---------------------------------------------------------------------------------------------------------
+struct QkvConvArgs {
+    const float* proj;       // [T, ld]
+    int ld, col0;
+    const float* w;          // [taps][C]
+    int taps, C;
+    float* state;            // [slots][(taps - 1) * C] or null when taps == 1
+    long long state_stride;
+    const int* positions;
+    const int* row_req;
+    const int* row_offsets;
+    const int* state_slots;
+    const int* block_table;
+    const float* inv_freq;   // [rot / 2] or null
+    void* q_out;             // [T, nq, D]
+    void* kv_base;           // [page][2][nkv][page_size][D]
+    int T, nq, nkv, D, dk, dv, rot, pairing;
+    int max_blocks, page_size;
+};
+
+template <int VEC> __device__ __forceinline__ void read_vec(const float* p, float* v) {
+    if (VEC == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        v[0] = x.x; v[1 % VEC] = x.y; v[2 % VEC] = x.z; v[3 % VEC] = x.w;
+    } else {
+        v[0] = *p;
+    }
+}
+template <typename TO, int VEC> __device__ __forceinline__ void write_vec(TO* p, const float* v) {
+    if (VEC == 4) store4<TO>(p, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
+    else *p = from_float<TO>(v[0]);
+}
+
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(256) qkv_conv_kernel(QkvConvArgs a) {
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int slots = a.nq + 2 * a.nkv;
+    const long long work = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
+    if (work >= (long long)a.T * slots) return;
+    const int t = (int)(work / slots), slot = (int)(work % slots);
+    const int b = a.row_req[t];
+    const int first = a.row_offsets[b], n = a.row_offsets[b + 1] - first;
+    const int i0 = t - first;                                  // place within the portion
+    const int keep = a.taps - 1;
+    if (i0 > 0 && i0 < keep) return;                           // served by the portion's first row
+    const bool lead = i0 == 0 && keep > 0;
+    const int count = lead ? min(keep, n) : 1;
+    const bool is_q = slot < a.nq;
+    const bool is_v = slot >= a.nq + a.nkv;
+    const int size = is_v ? a.dv : a.dk;                       // the head's own elements; zeros behind, up to D
+    const int ch0 = is_q ? slot * a.dk : is_v ? (a.nq + a.nkv) * a.dk + (slot - a.nq - a.nkv) * a.dv : slot * a.dk;
+    const int rot = is_v ? 0 : a.rot, half = rot >> 1;
+    const float* in = a.proj + a.col0 + ch0;
+    const float* w = a.w + ch0;
+    float* st = keep > 0 ? a.state + (size_t)a.state_slots[b] * a.state_stride + ch0 : nullptr;
+    const size_t plane = (size_t)a.nkv * a.page_size * a.D;
+    for (int r = 0; r < count; ++r) {
+        const int i = i0 + r, row = t + r;
+        const int pos = a.positions[row];
+        TO* dst;
+        if (is_q) {
+            dst = (TO*)a.q_out + ((size_t)row * a.nq + slot) * a.D;
+        } else {
+            const int head = is_v ? slot - a.nq - a.nkv : slot - a.nq;
+            const int page = a.block_table[(size_t)b * a.max_blocks + pos / a.page_size];
+            if (page < 0) continue;                            // the host checks that written positions have pages
+            dst = (TO*)a.kv_base + ((size_t)page * 2 + (is_v ? 1 : 0)) * plane +
+                  ((size_t)head * a.page_size + (pos % a.page_size)) * a.D;
+        }
+        auto conv = [&](int e, float* y) {                     // elements e .. e + VEC - 1 of the head after the convolution
+            float acc[VEC];
+#pragma unroll
+            for (int u = 0; u < VEC; ++u) acc[u] = 0.0f;
+            for (int j = 0; j < a.taps; ++j) {
+                const int back = keep - j;
+                float x[VEC], ww[VEC];
+                read_vec<VEC>(w + (size_t)j * a.C + e, ww);
+                if (i >= back) read_vec<VEC>(in + (size_t)(row - back) * a.ld + e, x);
+                else read_vec<VEC>(st + (size_t)(i + j) * a.C + e, x);
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) acc[u] = fmaf(ww[u], x[u], acc[u]);
+            }
+#pragma unroll
+            for (int u = 0; u < VEC; ++u) y[u] = acc[u];
+        };
+        for (int e = lane * VEC; e < a.D; e += 32 * VEC) {
+            float y[VEC];
+            if (e >= size) {
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) y[u] = 0.0f;
+                write_vec<TO, VEC>(dst + e, y);
+            } else if (e >= rot) {
+                conv(e, y);
+                write_vec<TO, VEC>(dst + e, y);
+            } else if (e < half) {                             // with VEC = 4: halves layout, half a multiple of 4
+                float z[VEC];
+                const int e0 = a.pairing == ROPE_HALVES ? e : 2 * e, e1 = a.pairing == ROPE_HALVES ? e + half : 2 * e + 1;
+                conv(e0, y);
+                conv(e1, z);
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) {
+                    float sn, cs;
+                    sincosf((float)pos * a.inv_freq[e + u], &sn, &cs);
+                    const float y0 = y[u] * cs - z[u] * sn, z0 = z[u] * cs + y[u] * sn;
+                    y[u] = y0;
+                    z[u] = z0;
+                }
+                write_vec<TO, VEC>(dst + e0, y);
+                write_vec<TO, VEC>(dst + e1, z);
+            }
+        }
+    }
+    if (!lead) return;
+    __syncwarp();                                              // every lane has read the old state
+    for (int e = lane; e < size; e += 32)
+        for (int j = 0; j < keep; ++j) {                       // ascending: place j + n is read before it is overwritten
+            const int src = n - keep + j;
+            st[(size_t)j * a.C + e] = src >= 0 ? in[(size_t)(first + src) * a.ld + e] : st[(size_t)(j + n) * a.C + e];
+        }
+}
+
+SHARPI_API int sharpi_qkv_conv(const float* proj, int ld, int col0, const float* w, int taps, float* state,
+                               long long state_stride, const int* positions, const int* row_req, const int* row_offsets,
+                               const int* state_slots, const int* block_table, const float* inv_freq, int rot, int pairing,
+                               void* q_out, void* kv_base, int out_dtype, int T, int nq, int nkv, int D, int dk, int dv,
+                               int max_blocks, int page_size, cudaStream_t stream) {
+    if (T <= 0) return SHARPI_OK;
+    if (nq <= 0 || nkv <= 0 || D <= 0 || dk <= 0 || dk > D || dv <= 0 || dv > D || page_size <= 0 || max_blocks <= 0 ||
+        taps <= 0 || (taps > 1 && !state) || !w)
+        return SHARPI_BAD_ARGUMENT;
+    if (rot < 0 || (rot & 1) || rot > dk || (rot && !inv_freq)) return SHARPI_BAD_ARGUMENT;
+    if (pairing != ROPE_INTERLEAVED && pairing != ROPE_HALVES) return SHARPI_BAD_ARGUMENT;
+    QkvConvArgs a;
+    a.C = (nq + nkv) * dk + nkv * dv;
+    if (col0 < 0 || col0 + a.C > ld) return SHARPI_BAD_ARGUMENT;
+    a.proj = proj; a.ld = ld; a.col0 = col0; a.w = w; a.taps = taps; a.state = state; a.state_stride = state_stride;
+    a.positions = positions; a.row_req = row_req; a.row_offsets = row_offsets; a.state_slots = state_slots;
+    a.block_table = block_table; a.inv_freq = inv_freq; a.q_out = q_out; a.kv_base = kv_base;
+    a.T = T; a.nq = nq; a.nkv = nkv; a.D = D; a.dk = dk; a.dv = dv; a.rot = rot; a.pairing = pairing;
+    a.max_blocks = max_blocks; a.page_size = page_size;
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(state) |
+                           reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(kv_base);
+    const bool vec = dk % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && (rot / 2) % 4 == 0 &&
+                     (rot == 0 || pairing == ROPE_HALVES) && state_stride % 4 == 0 && (ptrs & 15) == 0;
+    const long long work = (long long)T * (nq + 2 * nkv);
+    const long long blocks = (work + 7) / 8;
+    if (blocks > 2147483647LL) return SHARPI_BAD_ARGUMENT;
+#define CONV_CASE(TO, V)                                                       \
+    do {                                                                       \
+        auto kern = qkv_conv_kernel<TO, V>;                                    \
+        SHARPI_LAUNCH_PDL(kern, (unsigned)blocks, 256, 0, stream, a);          \
+    } while (0)
+    if (out_dtype == SHARPI_F32) { if (vec) CONV_CASE(float, 4); else CONV_CASE(float, 1); }
+    else if (out_dtype == SHARPI_BF16) { if (vec) CONV_CASE(bf16, 4); else CONV_CASE(bf16, 1); }
+    else return SHARPI_BAD_ARGUMENT;
+#undef CONV_CASE
+    return SHARPI_OK;
+}

@@ -50,6 +50,7 @@ struct TcGemmParams {
     int* status;                // device word: 0 ok, else the code of the wait that gave up
     int rows, N, K, E;          // N: weight rows per expert (MODE_SWIGLU: 2 I)
     int accumulate;
+    float gate_limit;           // MODE_SWIGLU: > 0 = the clamped gate with this limit in place of silu(g) * u
     int store_act;              // MODE_STORE: 0 = float32 out as above; 1 / 2 / 3 = bf16 out [rows, N] (sorted rows) of
                                 // relu(x)^2 / tanh-GELU(x) / SiLU(x): the first product of a two-layer expert
     // K split over gridDim.z CTAs (few rows and few experts: not enough tiles to fill the GPU otherwise).
@@ -94,6 +95,13 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
     return g * rcp_approx(1.0f + ex2_approx(-1.4426950408889634f * g)) * u;
 }
 
+// The clamped form: g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
+__device__ __forceinline__ float clamped_gate_mul(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * rcp_approx(1.0f + ex2_approx(-1.702f * 1.4426950408889634f * g)) * (u + 1.0f);
+}
+
 __device__ __forceinline__ float store_activation(int kind, float x) {
     if (kind == 1) { const float r = fmaxf(x, 0.0f); return r * r; }
     if (kind == 2) return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
@@ -124,7 +132,8 @@ __device__ __forceinline__ void tc_epilogue_chunk(const TcGemmParams& p, const f
             for (int j = 0; j < 16; ++j) {
                 if (j < count) {
                     const float gv = g[j] * sc[j], uv = u[j] * sc[j];
-                    act[(size_t)(r_first + j) * I + n] = __float2bfloat16_rn(silu_mul(gv, uv));
+                    act[(size_t)(r_first + j) * I + n] =
+                        __float2bfloat16_rn(p.gate_limit > 0.0f ? clamped_gate_mul(gv, uv, p.gate_limit) : silu_mul(gv, uv));
                 }
             }
         }
@@ -735,7 +744,7 @@ static int tc_grouped_gemm_impl(const void* A, const void* W, const int* group_o
                                const int* out_rows, const float* row_scale, const int* scale_rows,
                                int* status, float* partial, int* tickets, int rows, int N, int K, int E, int mode,
                                int row_tile, int accumulate, int k_split, int max_ctas, int store_act,
-                               cudaStream_t stream) {
+                               float gate_limit, cudaStream_t stream) {
     if (rows <= 0 || N <= 0) return SHARPI_OK;
     if (store_act < 0 || store_act > 3 || (store_act && (mode != MODE_STORE || accumulate || out_rows)))
         return SHARPI_BAD_ARGUMENT;
@@ -751,6 +760,8 @@ static int tc_grouped_gemm_impl(const void* A, const void* W, const int* group_o
     p.group_offsets = group_offsets; p.out_rows = out_rows; p.row_scale = row_scale; p.scale_rows = scale_rows;
     p.out = out; p.status = status; p.rows = rows; p.N = N; p.K = K; p.E = E; p.accumulate = accumulate;
     p.store_act = store_act;
+    if (!(gate_limit >= 0.0f)) return SHARPI_BAD_ARGUMENT;
+    p.gate_limit = gate_limit;
     if (k_split < 1 || k_split > 16 || (k_split > 1 && (!partial || !tickets))) return SHARPI_BAD_ARGUMENT;
     p.partial = partial; p.k_split = k_split; p.tickets = tickets;
     p.wait_limit = g_test_wait_limit ? g_test_wait_limit : WAIT_LIMIT;
@@ -794,7 +805,7 @@ SHARPI_API int sharpi_tc_grouped_gemm(const void* A, const void* W, const int* g
                                       int* status, float* partial, int* tickets, int rows, int N, int K, int E, int mode,
                                       int row_tile, int accumulate, int k_split, int max_ctas, cudaStream_t stream) {
     return tc_grouped_gemm_impl(A, W, group_offsets, out, out_rows, row_scale, scale_rows, status, partial, tickets, rows,
-                                N, K, E, mode, row_tile, accumulate, k_split, max_ctas, 0, stream);
+                                N, K, E, mode, row_tile, accumulate, k_split, max_ctas, 0, 0.0f, stream);
 }
 
 // The store mode with an activation in the epilogue: bf16 out[r, n] = act(a[r] . w[e(r)][n]) in sorted row order
@@ -804,7 +815,17 @@ SHARPI_API int sharpi_tc_grouped_gemm_act(const void* A, const void* W, const in
                                           int row_tile, int k_split, int act, cudaStream_t stream) {
     if (act < 1 || act > 3) return SHARPI_BAD_ARGUMENT;
     return tc_grouped_gemm_impl(A, W, group_offsets, out, nullptr, nullptr, nullptr, status, partial, tickets, rows, N, K,
-                                E, MODE_STORE, row_tile, 0, k_split, 0, act, stream);
+                                E, MODE_STORE, row_tile, 0, k_split, 0, act, 0.0f, stream);
+}
+
+// The gate|up mode with the clamped gate in the epilogue: bf16 out[r, i] = g sigmoid(1.702 g) (u + 1) with g cut off above
+// at `limit` and u on both sides, in sorted row order.
+SHARPI_API int sharpi_tc_grouped_gemm_clamped(const void* A, const void* W, const int* group_offsets, void* out,
+                                              int* status, float* partial, int* tickets, int rows, int N, int K, int E,
+                                              int row_tile, int k_split, float limit, cudaStream_t stream) {
+    if (!(limit > 0.0f)) return SHARPI_BAD_ARGUMENT;
+    return tc_grouped_gemm_impl(A, W, group_offsets, out, nullptr, nullptr, nullptr, status, partial, tickets, rows, N, K,
+                                E, MODE_SWIGLU, row_tile, 0, k_split, 0, 0, limit, stream);
 }
 
 // out[r, :] = in[rows[r], :] for bf16 rows of width K (a multiple of 8): the activations sorted by

@@ -69,10 +69,12 @@ class StepRunner:
         # step's one metadata copy; it knows nothing of what they mean.
         self.planners: Dict[Hashable, object] = {}
         for b in getattr(model, "blocks", []):
-            make = getattr(b.mixer, "step_planner", None)
-            planner = make(cache.page_size) if make is not None else None
-            if planner is not None:
-                self.planners.setdefault(planner.key, planner)
+            several = getattr(b.mixer, "step_planners", None)
+            one = getattr(b.mixer, "step_planner", None)
+            made = several(cache.page_size) if several is not None else [one(cache.page_size)] if one is not None else []
+            for planner in made:
+                if planner is not None:
+                    self.planners.setdefault(planner.key, planner)
         self.steps_run = 0
         self.rows_run = 0
         # Tracing, for hunting the first difference: when `trace_router` is set, every routed

@@ -84,6 +84,17 @@ SIGNATURES: Dict[str, Tuple[str, list]] = {
     "sharpi_ssd_scan": ("mamba2", [P, I, I, I, I, P, I, I, P, P, P, P, P, P, LL, P, I, I, I, I, I, I, P]),
     "sharpi_add_layernorm": ("elementwise", [P, P, P, P, F, P, I, I, P, I, P, P]),
     "sharpi_qkv_post_wide": ("rope_kv", [P, I, P, P, P, P, P, F, I, I, P, P, I, I, I, I, I, I, I, F, F, I, I, P]),
+    "sharpi_add_rmsnorm_pair": ("elementwise", [P, P, P, P, F, I, I, P, P, I, P, P]),
+    "sharpi_gated_cols": ("elementwise", [P, P, P, I, I, I, I, I, I, I, F, P]),
+    "sharpi_gate_heads": ("elementwise", [P, P, I, P, I, I, I, I, I, I, F, P]),
+    "sharpi_softcap": ("elementwise", [P, F, LL, P]),
+    "sharpi_qkv_conv": ("rope_kv", [P, I, I, P, I, P, LL, P, P, P, P, P, P, I, I, P, P, I, I, I, I, I, I, I, I, I, P]),
+    "sharpi_lightning_walk": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, LL, P, I, I, I, P]),
+    "sharpi_lightning_chunks": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, I, P, P, LL, P, I, I, I, P]),
+    "sharpi_norm_sigmoid_gate": ("lightning", [P, P, I, P, F, F, I, I, P, I, I, P]),
+    "sharpi_router_groups": ("moe_topk", [P, P, P, I, I, I, I, F, I, I, I, P, P, P, P, P, P]),
+    "sharpi_moe_combine_full": ("moe_topk", [P, P, P, P, P, P, P, P, I, I, I, I, P]),
+    "sharpi_tc_grouped_gemm_clamped": ("tc_gemm", [P, P, P, P, P, P, P, I, I, I, I, I, I, F, P]),
     "sharpi_gated_group_norm": ("mamba2", [P, P, I, P, F, I, I, I, P, I, P]),
 }
 

@@ -1493,3 +1493,273 @@ def qkv_post_wide(qkv: torch.Tensor, positions: torch.Tensor, row_req: torch.Ten
                                          dtype_code(q_out.dtype), T, nq, nkv, d, block_table.shape[-1], page_size,
                                          float(temp_coef), float(temp_every), int(write_kv), int(has_kv), _stream()),
           "sharpi_qkv_post_wide")
+
+
+# ---------------------------------------------------------------------------------------
+# two norms of one stream, gated activations into column ranges, head gates, capped logits
+# ---------------------------------------------------------------------------------------
+def add_rmsnorm_pair(x: torch.Tensor, delta: Optional[torch.Tensor], w1: torch.Tensor, w2: torch.Tensor, eps: float,
+                     out_dtype: torch.dtype, *, want_fp32: bool = False):
+    """:func:`add_rmsnorm` under two weights at once: ``x += delta`` in place, then the normalised row times ``w1`` and times
+    ``w2``.  Returns ``(out1, out2, out2 in float32 or None)``."""
+    _need(x, "x", torch.float32)
+    _need(w1, "w1", torch.float32)
+    _need(w2, "w2", torch.float32)
+    T, H = x.shape
+    if w1.numel() != H or w2.numel() != H:
+        raise KernelError(f"norm weights have {w1.numel()} and {w2.numel()} entries, the rows have {H}")
+    if delta is not None:
+        _need(delta, "delta", torch.float32)
+        if delta.shape != x.shape:
+            raise KernelError(f"delta shape {tuple(delta.shape)} differs from x shape {tuple(x.shape)}")
+    out1 = torch.empty((T, H), dtype=out_dtype, device=x.device)
+    out2 = torch.empty((T, H), dtype=out_dtype, device=x.device)
+    out32 = None
+    if want_fp32:
+        out32 = out2 if out_dtype == torch.float32 else torch.empty((T, H), dtype=torch.float32, device=x.device)
+    check(kernel("sharpi_add_rmsnorm_pair")(x.data_ptr(), _ptr(delta), w1.data_ptr(), w2.data_ptr(), float(eps), T, H,
+                                            out1.data_ptr(), out2.data_ptr(), dtype_code(out_dtype),
+                                            None if out32 is out2 else _ptr(out32), _stream()), "sharpi_add_rmsnorm_pair")
+    return out1, out2, out32
+
+
+def gated_cols(gate_up: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None, act: int = ACT_SILU,
+               limit: float = 0.0, ones: int = 0) -> torch.Tensor:
+    """The gated activation of a fused gate|up product ``[M, 2I]`` (float32) into ``out``, a column range ``[M, n]`` of a
+    possibly wider matrix, ``n >= I``: ``act(g) * u`` with ``bias`` (float32 ``[2I]``) added to g and u first, or, with
+    ``limit`` > 0, ``g sigmoid(1.702 g) (u + 1)`` with g cut off above at ``limit`` and u on both sides.  Columns behind
+    the first I become ``ones`` columns of 1 and then zeros."""
+    _need(gate_up, "gate_up", torch.float32)
+    ld = _need_columns(out, "out")
+    M, I2 = gate_up.shape
+    I = I2 // 2
+    if out.shape[0] != M or out.shape[1] < I + ones:
+        raise KernelError(f"out is {tuple(out.shape)} for {M} rows of {I} elements and {ones} columns of ones")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != I2:
+            raise KernelError(f"bias has {bias.numel()} entries, the rows have {I2}")
+    check(kernel("sharpi_gated_cols")(gate_up.data_ptr(), _ptr(bias), out.data_ptr(), dtype_code(out.dtype), M, I, ld,
+                                      int(ones), out.shape[1] - I - int(ones), int(act), float(limit), _stream()),
+          "sharpi_gated_cols")
+    return out
+
+
+def gate_heads(o: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, *, heads: int, D: int, dv: int,
+               scale: float = 1.0) -> torch.Tensor:
+    """``out[t, h dv + i] = o[t, h, i] * sigmoid(gate[t, h]) * scale``: heads ``D`` elements apart in ``o``, side by side in
+    the column range ``out`` ``[T, heads * dv]``; ``gate`` float32 ``[T, heads]`` (a column range too)."""
+    _need(o, "o")
+    ld_g, ld_o = _need_columns(gate, "gate", torch.float32), _need_columns(out, "out", o.dtype)
+    T = gate.shape[0]
+    if o.numel() != T * heads * D or tuple(out.shape) != (T, heads * dv) or gate.shape[1] != heads:
+        raise KernelError(f"shapes disagree: o {tuple(o.shape)}, gate {tuple(gate.shape)}, out {tuple(out.shape)}")
+    check(kernel("sharpi_gate_heads")(o.data_ptr(), gate.data_ptr(), ld_g, out.data_ptr(), ld_o, dtype_code(o.dtype), T,
+                                      heads, D, dv, float(scale), _stream()), "sharpi_gate_heads")
+    return out
+
+
+def softcap_(y: torch.Tensor, cap: float) -> torch.Tensor:
+    """``y = cap * tanh(y / cap)`` in place (float32)."""
+    _need(y, "y", torch.float32)
+    check(kernel("sharpi_softcap")(y.data_ptr(), float(cap), y.numel(), _stream()), "sharpi_softcap")
+    return y
+
+
+# ---------------------------------------------------------------------------------------
+# short convolutions on q, k and v
+# ---------------------------------------------------------------------------------------
+def qkv_conv(proj: torch.Tensor, q_out: torch.Tensor, kv_layer: torch.Tensor, *, weight: torch.Tensor,
+             state: Optional[torch.Tensor], positions: torch.Tensor, row_req: torch.Tensor, row_offsets: torch.Tensor,
+             state_slots: torch.Tensor, block_table: torch.Tensor, nq: int, nkv: int, D: int, key_dim: int, value_dim: int,
+             page_size: int, inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0, pairing: int = ROPE_HALVES) -> None:
+    """Causal convolution of every channel of q | k | v (``proj`` float32 ``[T, C]``, a column range of a wider product, heads
+    unpadded), rotation of the first ``rot_dims`` elements of q and k, q store (``q_out`` ``[T, nq, D]``, zeros behind
+    ``key_dim``) and the scatter of k and v into pages.  ``weight`` float32 ``[taps, C]``; ``state`` float32
+    ``[slots, (taps - 1) * C]``, read and moved on."""
+    ld = _need_columns(proj, "proj", torch.float32)
+    _need(weight, "weight", torch.float32)
+    _need(q_out, "q_out")
+    _need(kv_layer, "kv_layer", q_out.dtype)
+    for name, t in (("positions", positions), ("row_req", row_req), ("row_offsets", row_offsets),
+                    ("state_slots", state_slots), ("block_table", block_table)):
+        _need(t, name, torch.int32)
+    T, C = positions.numel(), (nq + nkv) * key_dim + nkv * value_dim
+    taps = weight.shape[0]
+    if tuple(proj.shape) != (T, C) or weight.shape[1] != C:
+        raise KernelError(f"proj is {tuple(proj.shape)} and weight {tuple(weight.shape)} for [T={T}, C={C}]")
+    if tuple(kv_layer.shape[1:]) != (2, nkv, page_size, D) or tuple(q_out.shape) != (T, nq, D):
+        raise KernelError(f"kv_layer is {tuple(kv_layer.shape)}, q_out {tuple(q_out.shape)}")
+    if taps > 1:
+        _need(state, "state", torch.float32)
+        if state[0].numel() != (taps - 1) * C:
+            raise KernelError(f"state rows hold {state[0].numel()} floats, expected {(taps - 1) * C}")
+    if rot_dims:
+        _need(inv_freq, "inv_freq", torch.float32)
+        if inv_freq.numel() != rot_dims // 2:
+            raise KernelError(f"{rot_dims} rotated elements need {rot_dims // 2} frequencies, found {inv_freq.numel()}")
+    check(kernel("sharpi_qkv_conv")(proj.data_ptr(), ld, 0, weight.data_ptr(), taps, _ptr(state) if taps > 1 else None,
+                                    state.stride(0) if taps > 1 else 0, positions.data_ptr(), row_req.data_ptr(),
+                                    row_offsets.data_ptr(), state_slots.data_ptr(), block_table.data_ptr(),
+                                    _ptr(inv_freq) if rot_dims else None, int(rot_dims), int(pairing), q_out.data_ptr(),
+                                    kv_layer.data_ptr(), dtype_code(q_out.dtype), T, nq, nkv, D, key_dim, value_dim,
+                                    block_table.shape[-1], page_size, _stream()), "sharpi_qkv_conv")
+
+
+# ---------------------------------------------------------------------------------------
+# linear attention with a constant decay per head
+# ---------------------------------------------------------------------------------------
+LIGHTNING_CHUNK = 64
+LIGHTNING_MAX_KEY = 512
+
+
+def decay_powers(decay) -> torch.Tensor:
+    """float32 ``[heads, LIGHTNING_CHUNK + 1]``: the powers ``a^0 .. a^chunk`` of every head's decay, formed in float64."""
+    a = torch.as_tensor([float(x) for x in decay], dtype=torch.float64).view(-1, 1)
+    return torch.pow(a, torch.arange(LIGHTNING_CHUNK + 1, dtype=torch.float64).view(1, -1)).to(torch.float32).contiguous()
+
+
+def lightning(proj: torch.Tensor, *, col_q: int, col_k: int, col_v: int, powers: torch.Tensor, row_offsets: torch.Tensor,
+              state_slots: torch.Tensor, state: torch.Tensor, heads: int, d: int, dv: int, num_requests: int,
+              walk_requests: Optional[torch.Tensor] = None, num_walk: Optional[int] = None,
+              chunks: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``S <- a S + silu(k) silu(v)^T``, ``o = S^T silu(q)`` per head for the step's rows; float32 ``[T, heads * dv]``.
+    ``proj`` float32 ``[T, *]`` (a column range) holds q, k and v at the named columns; ``state`` float32
+    ``[slots, heads * d * dv]``.  ``walk_requests`` (None: all ``num_requests``) are walked row by row; the requests of
+    ``spans`` (int32 ``[m, 4]``) by chunks (int32 ``[n, 4]``, at most LIGHTNING_CHUNK rows each)."""
+    ld = _need_columns(proj, "proj", torch.float32)
+    _need(powers, "powers", torch.float32)
+    _need(state, "state", torch.float32)
+    _need(row_offsets, "row_offsets", torch.int32)
+    _need(state_slots, "state_slots", torch.int32)
+    T = proj.shape[0]
+    if tuple(powers.shape) != (heads, LIGHTNING_CHUNK + 1):
+        raise KernelError(f"powers is {tuple(powers.shape)}, expected {(heads, LIGHTNING_CHUNK + 1)}")
+    if state[0].numel() != heads * d * dv or max(col_q + heads * d, col_k + heads * d, col_v + heads * dv) > proj.shape[1]:
+        raise KernelError(f"state rows hold {state[0].numel()} floats and proj {proj.shape[1]} columns for {heads} heads of "
+                          f"{d} x {dv}")
+    y = torch.empty((T, heads * dv), dtype=torch.float32, device=proj.device)
+    n_walk = num_requests if num_walk is None else int(num_walk)
+    if chunks is not None:
+        _need(chunks, "chunks", torch.int32)
+        _need(spans, "spans", torch.int32)
+        sums = torch.empty((chunks.shape[0], heads, d, dv), dtype=torch.float32, device=proj.device)
+        check(kernel("sharpi_lightning_chunks")(proj.data_ptr(), ld, col_q, col_k, col_v, powers.data_ptr(),
+                                                row_offsets.data_ptr(), state_slots.data_ptr(), chunks.data_ptr(),
+                                                chunks.shape[0], spans.data_ptr(), spans.shape[0], sums.data_ptr(),
+                                                state.data_ptr(), state.stride(0), y.data_ptr(), heads, d, dv, _stream()),
+              "sharpi_lightning_chunks")
+    if n_walk:
+        if walk_requests is not None:
+            _need(walk_requests, "walk_requests", torch.int32)
+        check(kernel("sharpi_lightning_walk")(proj.data_ptr(), ld, col_q, col_k, col_v, powers.data_ptr(),
+                                              row_offsets.data_ptr(), state_slots.data_ptr(), _ptr(walk_requests), n_walk,
+                                              state.data_ptr(), state.stride(0), y.data_ptr(), heads, d, dv, _stream()),
+              "sharpi_lightning_walk")
+    return y
+
+
+def norm_sigmoid_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, *,
+                      scale: float = 1.0) -> torch.Tensor:
+    """``out = y / sqrt(mean(y^2) + eps) * weight * sigmoid(gate) * scale`` over whole rows; ``y`` float32 ``[T, n]``, ``gate``
+    float32 and ``out`` column ranges ``[T, n]``."""
+    _need(y, "y", torch.float32)
+    _need(weight, "weight", torch.float32)
+    ld_g, ld_o = _need_columns(gate, "gate", torch.float32), _need_columns(out, "out")
+    T, n = y.shape
+    if tuple(gate.shape) != (T, n) or tuple(out.shape) != (T, n) or weight.numel() != n:
+        raise KernelError(f"shapes disagree: y {tuple(y.shape)}, gate {tuple(gate.shape)}, out {tuple(out.shape)}, weight "
+                          f"{weight.numel()}")
+    check(kernel("sharpi_norm_sigmoid_gate")(y.data_ptr(), gate.data_ptr(), ld_g, weight.data_ptr(), float(eps), float(scale),
+                                             T, n, out.data_ptr(), ld_o, dtype_code(out.dtype), _stream()),
+          "sharpi_norm_sigmoid_gate")
+    return out
+
+
+# ---------------------------------------------------------------------------------------
+# mixtures routed by a softmax over all experts, in groups, with identity experts
+# ---------------------------------------------------------------------------------------
+def router_groups(h32: torch.Tensor, router_weight: torch.Tensor, k: int, *, correction: Optional[torch.Tensor] = None,
+                  scale: float = 1.0, renormalize: bool = True, n_groups: int = 1, keep: int = 1,
+                  gate_weight: Optional[torch.Tensor] = None, want_scores: bool = False):
+    """``s = softmax(h . Wr^T)`` in float32; the ``k`` largest of ``s + correction`` among the experts of the ``keep`` best of
+    ``n_groups`` groups of neighbours (a group's score is its largest ``s + correction``); weights ``scale * s``, divided by
+    the chosen ``s``' sum + 1e-20 first when ``renormalize``.  ``gate_weight`` float32 ``[H]``: also
+    ``sigmoid(gate_weight . h)`` per row.  Returns ``(expert int32 [T, k], weight float32 [T, k], gate [T] or None, scores
+    [T, E] or None)``."""
+    _need(h32, "h32", torch.float32)
+    _need(router_weight, "router_weight", torch.float32)
+    T, H = h32.shape
+    E = router_weight.shape[0]
+    if router_weight.shape[1] != H:
+        raise KernelError(f"router weight is {tuple(router_weight.shape)}, activations have width {H}")
+    if correction is not None:
+        _need(correction, "correction", torch.float32)
+        if correction.numel() != E:
+            raise KernelError(f"correction has {correction.numel()} entries for {E} experts")
+    if n_groups < 1 or E % n_groups or not (1 <= keep <= n_groups) or not (1 <= k <= min(keep * (E // n_groups), 32)):
+        raise KernelError(f"{k} of {E} experts in {n_groups} groups of which {keep} are kept")
+    if gate_weight is not None:
+        _need(gate_weight, "gate_weight", torch.float32)
+        if gate_weight.numel() != H:
+            raise KernelError(f"gate weight has {gate_weight.numel()} entries, activations have width {H}")
+    expert = torch.empty((T, k), dtype=torch.int32, device=h32.device)
+    weight = torch.empty((T, k), dtype=torch.float32, device=h32.device)
+    gate = torch.empty((T,), dtype=torch.float32, device=h32.device) if gate_weight is not None else None
+    scores = torch.empty((T, E), dtype=torch.float32, device=h32.device) if want_scores else None
+    check(kernel("sharpi_router_groups")(h32.data_ptr(), router_weight.data_ptr(), _ptr(correction), T, H, E, k,
+                                         float(scale), int(renormalize), int(n_groups), int(keep), _ptr(gate_weight),
+                                         _ptr(gate), expert.data_ptr(), weight.data_ptr(), _ptr(scores), _stream()),
+          "sharpi_router_groups")
+    return expert, weight, gate, scores
+
+
+def moe_combine_full(y_pairs: torch.Tensor, expert: torch.Tensor, weight: torch.Tensor, h32: torch.Tensor, num_experts: int, *,
+                     shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                     add: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[t] = add[t] + gate[t] shared[t] + sum_j (y_pairs[t k + j], or weight[t, j] h32[t] where expert[t, j] >=
+    num_experts)`` (float32, the choices in their order).  ``y_pairs`` holds products that already carry their weight."""
+    _need(y_pairs, "y_pairs", torch.float32)
+    _need(expert, "expert", torch.int32)
+    _need(weight, "weight", torch.float32)
+    _need(h32, "h32", torch.float32)
+    (T, k), H = expert.shape, h32.shape[1]
+    if tuple(y_pairs.shape) != (T * k, H) or h32.shape[0] != T:
+        raise KernelError(f"y_pairs is {tuple(y_pairs.shape)}, expected {(T * k, H)}")
+    for name, t, shape in (("shared", shared, (T, H)), ("add", add, (T, H)), ("gate", gate, (T,))):
+        if t is not None:
+            _need(t, name, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"{name} is {tuple(t.shape)}, expected {shape}")
+    if out is None:
+        out = torch.empty((T, H), dtype=torch.float32, device=h32.device)
+    check(kernel("sharpi_moe_combine_full")(y_pairs.data_ptr(), expert.data_ptr(), weight.data_ptr(), h32.data_ptr(),
+                                            _ptr(shared), _ptr(gate), _ptr(add), out.data_ptr(), T, int(num_experts), k, H,
+                                            _stream()), "sharpi_moe_combine_full")
+    return out
+
+
+def tc_grouped_gemm_clamped(a: torch.Tensor, w: torch.Tensor, group_offsets: torch.Tensor, limit: float) -> torch.Tensor:
+    """The gate|up product of :func:`tc_grouped_gemm` with the clamped gate in its epilogue: bfloat16 ``out[r] = g
+    sigmoid(1.702 g) (u + 1)``, ``g`` cut off above at ``limit`` and ``u`` on both sides, in sorted row order."""
+    _need(a, "a", torch.bfloat16)
+    _need(w, "w", torch.bfloat16)
+    _need(group_offsets, "group_offsets", torch.int32)
+    rows, K = a.shape
+    E, N, Kw = w.shape
+    if Kw != K or group_offsets.numel() != E + 1:
+        raise KernelError(f"shapes disagree: a {tuple(a.shape)}, w {tuple(w.shape)}, offsets {group_offsets.numel()}")
+    if K % 8 != 0:
+        raise KernelError(f"the tensor-core product needs an inner size that is a multiple of 8, found {K}")
+    out = torch.empty((rows, N // 2), dtype=torch.bfloat16, device=a.device)
+    k_split = tc_k_split(rows, N // 2, sm_count(a.device))
+    partial = torch.empty((k_split, rows, N), dtype=torch.float32, device=a.device) if k_split > 1 else None
+    row_tile = tc_row_tile(rows, TC_MODE_SWIGLU, E)
+    tickets = None
+    if k_split > 1:
+        tickets = zeroed_tickets(a.device, ((N + 127) // 128) * (rows // max(row_tile, 1) + min(rows, E)))
+    check(kernel("sharpi_tc_grouped_gemm_clamped")(a.data_ptr(), w.data_ptr(), group_offsets.data_ptr(), out.data_ptr(),
+                                                   status_word(a.device).data_ptr(), _ptr(partial), _ptr(tickets), rows, N, K,
+                                                   E, row_tile, k_split, float(limit), _stream()),
+          "sharpi_tc_grouped_gemm_clamped")
+    return out

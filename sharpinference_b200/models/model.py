@@ -30,10 +30,11 @@ class DecoderModel:
     def __init__(self, *, embedding: torch.Tensor, blocks: Sequence[Block], final_norm: Norm, head: Linear,
                  act_dtype: torch.dtype, schedule: Optional[Sequence[ScheduleEntry]] = None,
                  eos_token_ids: Sequence[int] = (), config=None, stream_ops: Sequence[StreamOp] = (),
-                 embedder=None, logit_scale: float = 1.0, embedding_scale: float = 1.0):
+                 embedder=None, logit_scale: float = 1.0, embedding_scale: float = 1.0, logit_softcap: float = 0.0):
         """``embedder``: a part whose ``forward(ctx)`` gives the float32 residual stream(s) of the step's rows
         in place of the plain table lookup (its ``state_specs`` become per-request state of the model);
-        ``logit_scale`` multiplies the head's output, ``embedding_scale`` the looked-up embedding row."""
+        ``logit_scale`` multiplies the head's output, ``embedding_scale`` the looked-up embedding row;
+        ``logit_softcap`` > 0 turns a (scaled) logit ``y`` into ``cap * tanh(y / cap)``."""
         self.embedding = embedding                  # [V, H]
         self.blocks: List[Block] = list(blocks)
         self.stream_ops: List[StreamOp] = list(stream_ops)
@@ -49,6 +50,7 @@ class DecoderModel:
         self.state_specs = dict(getattr(embedder, "state_specs", None) or {})
         self.logit_scale = float(logit_scale)
         self.embedding_scale = float(embedding_scale)
+        self.logit_softcap = float(logit_softcap)
         self._validate_schedule()
 
     def set_schedule(self, schedule: Sequence[ScheduleEntry]) -> "DecoderModel":
@@ -105,4 +107,6 @@ class DecoderModel:
             return None
         h, _ = self.final_norm.apply(x, pending, rows=ctx.want_rows, out_dtype=self.act_dtype)
         logits = self.head(h)
-        return ops.scale_(logits, self.logit_scale) if self.logit_scale != 1.0 else logits
+        if self.logit_scale != 1.0:
+            logits = ops.scale_(logits, self.logit_scale)
+        return ops.softcap_(logits, self.logit_softcap) if self.logit_softcap > 0.0 else logits

@@ -201,8 +201,54 @@ class Mixer(Part):
         """The planner of this mixer's per-step metadata, or None if the step context is all it needs."""
         return None
 
+    def step_planners(self, page_size: int) -> List[StepPlanner]:
+        """All planners of this mixer: the one above, or several where a mixer is put together from mixers."""
+        planner = self.step_planner(page_size)
+        return [] if planner is None else [planner]
+
     def forward(self, ctx: StepContext, slot: LayerSlot, h: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
+
+
+class ColumnMixer(Mixer):
+    """A mixer that stands between two plain products: it reads columns of a projection of the layer's input and leaves
+    the columns that an output projection reads (``in_columns``, ``out_columns``).  Alone, :meth:`forward` runs both
+    products.  A part that holds several column mixers takes their weights over (:meth:`take_weights`), lays them side
+    by side, runs one product in front of all and one behind, and calls :meth:`inner`.
+
+    A subclass sets ``in_proj``, ``out_proj`` (``Linear``) and ``act_dtype`` and writes :meth:`inner`."""
+
+    in_columns: int
+    out_columns: int
+    in_proj: Any = None
+    out_proj: Any = None
+    act_dtype: torch.dtype = torch.bfloat16
+
+    def inner(self, ctx: StepContext, slot: LayerSlot, proj: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
+        """``proj`` float32 ``[T, in_columns]``, ``out`` ``[T, out_columns]`` in the activation dtype, either of them
+        possibly a column range of a wider matrix; ``out`` receives the mixer's columns times ``scale``."""
+        raise NotImplementedError
+
+    def inner_from(self, ctx: StepContext, slot: LayerSlot, h: torch.Tensor, out: torch.Tensor) -> None:
+        """From the layer's normalised input to the columns the output projection reads."""
+        self.inner(ctx, slot, self.in_proj(h), out)
+
+    def take_weights(self) -> Tuple[torch.Tensor, torch.Tensor]:
+        """Hand the input and the output weight over; :meth:`forward` does not work afterwards."""
+        w = (self.in_proj.weight, self.out_proj.weight)
+        self.in_proj = self.out_proj = None
+        return w
+
+    def take_out_weight(self) -> torch.Tensor:
+        """Hand the output weight over; the input product stays here (:meth:`inner_from`)."""
+        w = self.out_proj.weight
+        self.out_proj = None
+        return w
+
+    def forward(self, ctx: StepContext, slot: LayerSlot, h: torch.Tensor) -> torch.Tensor:
+        out = torch.empty((h.shape[0], self.out_columns), dtype=self.act_dtype, device=h.device)
+        self.inner_from(ctx, slot, h, out)
+        return self.out_proj(out)
 
 
 class FeedForward(Part):

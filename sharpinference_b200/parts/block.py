@@ -9,6 +9,11 @@ as ``pending`` and the next block's first norm (or the model's last) adds it.  A
 ``ParallelBlock`` has one norm whose output both sublayers read: ``h = norm(x)``,
 ``x += mixer(h) + ffn(h)``; the feed-forward may be absent.  The sum of the two outputs is the
 ``pending`` update.
+
+``ParallelPairBlock`` has two norms of the same stream: ``x += mixer(norm1(x)) + ffn(norm2(x))``.  Two RMS norms with one
+``eps`` are one kernel.  Where the mixer and the feed-forward both end in a plain product (a :class:`ColumnMixer` beside a
+feed-forward with ``out_columns``), their inner columns lie side by side in one matrix and one product forms the sum of
+both outputs.
 """
 from __future__ import annotations
 
@@ -17,7 +22,10 @@ from typing import Optional
 import torch
 
 from ..kernels import ops
-from .base import Block, FeedForward, LayerSlot, Mixer, Norm, StepContext, register_part
+from .base import Block, ColumnMixer, FeedForward, LayerSlot, Mixer, Norm, StepContext, register_part
+from .branches import side_by_side, pad_columns
+from .linear import Linear
+from .norm import RMSNorm
 
 
 @register_part("block", "prenorm")
@@ -52,3 +60,41 @@ class ParallelBlock(Block):
         if getattr(self.ffn, "adds_to", False):          # the feed-forward's last kernel adds the mixer's output in
             return x, self.ffn.forward(ctx, h, h32, add_to=mixed)
         return x, ops.add(mixed, self.ffn.forward(ctx, h, h32), out=mixed)
+
+
+@register_part("block", "parallel_pair")
+class ParallelPairBlock(Block):
+    def __init__(self, *, mixer_norm: Norm, mixer: Mixer, ffn_norm: Optional[Norm], ffn: Optional[FeedForward],
+                 act_dtype: torch.dtype = torch.bfloat16):
+        self.mixer_norm, self.mixer, self.ffn_norm, self.ffn, self.act_dtype = mixer_norm, mixer, ffn_norm, ffn, act_dtype
+        self._pair_norm = (isinstance(mixer_norm, RMSNorm) and isinstance(ffn_norm, RMSNorm)
+                           and mixer_norm.eps == ffn_norm.eps)
+        self.joint_out = None
+        if ffn is not None and isinstance(mixer, ColumnMixer) and hasattr(ffn, "take_out_weight"):
+            self.joint_out = Linear(side_by_side([mixer.take_out_weight(), ffn.take_out_weight()]), "mixer.o|mlp.down")
+            self._ffn_at = pad_columns(mixer.out_columns)
+
+    def _norms(self, x: torch.Tensor, pending: Optional[torch.Tensor], want32: bool):
+        if self._pair_norm:
+            return ops.add_rmsnorm_pair(x, pending, self.mixer_norm.weight, self.ffn_norm.weight, self.mixer_norm.eps,
+                                        self.act_dtype, want_fp32=want32)
+        h1, _ = self.mixer_norm.apply(x, pending, rows=None, out_dtype=self.act_dtype)
+        h2, h32 = self.ffn_norm.apply(x, None, rows=None, out_dtype=self.act_dtype, want_fp32=want32)
+        return h1, h2, h32
+
+    def forward(self, ctx: StepContext, slot: LayerSlot, x: torch.Tensor, pending: Optional[torch.Tensor]):
+        if self.ffn is None:
+            h, _ = self.mixer_norm.apply(x, pending, rows=None, out_dtype=self.act_dtype)
+            return x, self.mixer.forward(ctx, slot, h)
+        h1, h2, h32 = self._norms(x, pending, self.ffn.wants_fp32_input)
+        if self.joint_out is not None:
+            cols = torch.empty((x.shape[0], self.joint_out.in_features), dtype=self.act_dtype, device=x.device)
+            if self._ffn_at > self.mixer.out_columns:
+                cols[:, self.mixer.out_columns: self._ffn_at].zero_()
+            self.mixer.inner_from(ctx, slot, h1, cols[:, : self.mixer.out_columns])
+            self.ffn.inner(ctx, h2, cols[:, self._ffn_at:])
+            return x, self.joint_out(cols)
+        mixed = self.mixer.forward(ctx, slot, h1)
+        if getattr(self.ffn, "adds_to", False):
+            return x, self.ffn.forward(ctx, h2, h32, add_to=mixed)
+        return x, ops.add(mixed, self.ffn.forward(ctx, h2, h32), out=mixed)

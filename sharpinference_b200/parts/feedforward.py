@@ -1,6 +1,8 @@
 """Feed-forward parts: dense SwiGLU, a top-1 sigmoid-routed mixture of experts with an
 always-on shared expert, a dense two-layer network with a plain activation (``DenseMLP``) and a
-sigmoid-routed mixture in which every row uses k such networks (``MoESigmoidTopK``).
+sigmoid-routed mixture in which every row uses k such networks (``MoESigmoidTopK``), its gated form
+(``MoESigmoidTopKGated``), and a mixture routed by a softmax over all experts in groups, with identity experts, clamped
+gates and a gated shared expert (``MoESoftmaxGroups``).
 
 Dense (src/SharpInference.Engine/ForwardPass.cs:2006-2015): ``y = (silu(h Wg^T) * (h Wu^T)) Wd^T``.
 
@@ -26,19 +28,59 @@ from .linear import GroupedLinear, Linear
 class DenseSwiGLU(FeedForward):
     graph_safe = True        # reads the step through device tensors only: may be captured in a CUDA graph
     def __init__(self, *, gate_up: Linear, down: Linear, act_dtype: torch.dtype = torch.bfloat16,
-                 activation: str = "silu"):
-        """``activation``: what is applied to the gate half, ``silu`` (SwiGLU), ``gelu_tanh`` or ``relu2``."""
+                 activation: str = "silu", limit: float = 0.0):
+        """``activation``: what is applied to the gate half, ``silu`` (SwiGLU), ``gelu_tanh`` or ``relu2``.  ``limit`` > 0:
+        the clamped gate instead, ``g sigmoid(1.702 g) (u + 1)`` with g cut off above at ``limit`` and u on both sides.
+        Both projections may have biases; the first one's is added in the activation's kernel."""
         if gate_up.out_features != 2 * down.in_features:
             raise ValueError(f"fused gate|up weight has {gate_up.out_features} rows, expected 2 * {down.in_features}")
         if activation not in ops.ACTIVATIONS:
             raise ValueError(f"activation '{activation}' is not one of {', '.join(sorted(ops.ACTIVATIONS))}")
+        if limit < 0:
+            raise ValueError(f"the gate's limit must not be negative, found {limit}")
         self.gate_up, self.down, self.act_dtype, self.activation = gate_up, down, act_dtype, activation
+        self.limit = float(limit)
+        self.gate_up_bias = gate_up.bias
+        if gate_up.bias is not None:            # the activation's kernel adds it
+            self.gate_up = Linear(gate_up.weight, gate_up.name, stream_rows=gate_up.stream_rows)
+        self._bias_columns = 0
+
+    @property
+    def out_columns(self) -> int:
+        """Columns this network leaves for its last product, those that carry the product's bias included."""
+        n = self.gate_up.out_features // 2 + self._bias_columns
+        return (n + 7) // 8 * 8 if self._bias_columns else n
+
+    def take_out_weight(self) -> torch.Tensor:
+        """Hand the last product over to a part that forms it together with another one (:meth:`forward` does not work
+        afterwards): ``[H, out_columns]``.  A bias becomes columns of the weight that meet columns of ones in the
+        activations: one in float32; in bfloat16 three whose sum is the bias to 24 bits."""
+        w, bias = self.down.weight, self.down.bias
+        self.down = None
+        if bias is None:
+            return w
+        pieces, rest = [], bias.to(torch.float32)
+        for _ in range(1 if w.dtype == torch.float32 else 3):
+            pieces.append(rest.to(w.dtype))
+            rest = rest - pieces[-1].to(torch.float32)
+        self._bias_columns = len(pieces)
+        gap = self.out_columns - w.shape[1] - len(pieces)
+        zeros = torch.zeros((w.shape[0], gap), dtype=w.dtype, device=w.device)
+        return torch.cat([w, torch.stack(pieces, dim=1), zeros], dim=1).contiguous()
+
+    def inner(self, ctx: StepContext, h: torch.Tensor, out: torch.Tensor) -> None:
+        """The columns the last product reads, into ``out`` (the width may be padded: zeros behind)."""
+        ops.gated_cols(self.gate_up(h), out, bias=self.gate_up_bias, act=ops.ACTIVATIONS[self.activation], limit=self.limit,
+                       ones=self._bias_columns)
 
     def forward(self, ctx: StepContext, h: torch.Tensor, h32: Optional[torch.Tensor] = None,
                 out: Optional[torch.Tensor] = None, accumulate: bool = False) -> torch.Tensor:
-        if self.activation != "silu":
+        if self.gate_up_bias is not None or self.limit > 0:
+            act = torch.empty((h.shape[0], self.down.in_features), dtype=self.act_dtype, device=h.device)
+            self.inner(ctx, h, act)
+        elif self.activation != "silu":
             act = ops.gated_act(self.gate_up(h), ops.ACTIVATIONS[self.activation], self.act_dtype)
-        elif self.act_dtype == torch.bfloat16 and self.gate_up.streams(h) and self.gate_up.bias is None:
+        elif self.act_dtype == torch.bfloat16 and self.gate_up.streams(h):
             act = ops.dense_rows(h, self.gate_up.weight, swiglu=True)     # SwiGLU in the product's epilogue
         else:
             act = ops.swiglu(self.gate_up(h), self.act_dtype)
@@ -355,3 +397,96 @@ class MoESigmoidTopKGated(FeedForward):
         if side is not None:
             main.wait_stream(side)
         return ops.moe_combine(y, k, add=base, out=base)
+
+
+@register_part("feed_forward", "moe_softmax_groups")
+class MoESoftmaxGroups(FeedForward):
+    """A mixture of ``E`` gated experts and ``identity`` experts that hand their input on, of which every row uses
+    ``top_k``, with an optional shared expert that every row uses.
+
+    Router (float32, on the unrounded activations): ``s = softmax(Wr h)`` over all ``E + identity`` experts; choice score
+    ``s + correction``; the experts form ``groups`` equal groups of neighbours, only those of the ``keep`` groups with the
+    largest choice score in them can be chosen, and of these the ``top_k`` with the largest choice scores are (the lowest
+    index among equals).  Weights: the chosen ``s`` divided by their sum, times ``route_scale``.  An expert with weights
+    is ``W_down act(W_gate h, W_up h)`` without biases: SwiGLU, or with ``limit`` > 0 the clamped gate of
+    :class:`DenseSwiGLU`; an identity expert is ``h``.  The shared expert's output is multiplied by ``sigmoid(w . h)``
+    (``shared_gate`` ``[H]``; without it, by 1).
+
+    The gate of the shared expert is one more row of the router's kernel.  The (row, choice) pairs are sorted by expert
+    with the identity experts last, so that the grouped products (tcgen05 in bfloat16, the activation in the first one's
+    epilogue and the weight in the second one's) simply end before them; one kernel adds a row's pairs, its identity
+    terms, the shared expert and the mixer's output in a fixed order."""
+
+    wants_fp32_input = True
+    graph_safe = True
+    adds_to = True
+
+    def __init__(self, *, router: torch.Tensor, experts_gate_up: GroupedLinear, experts_down: GroupedLinear, top_k: int,
+                 identity: int = 0, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
+                 route_scale: float = 1.0, renormalize: bool = True, limit: float = 0.0,
+                 shared: Optional[DenseSwiGLU] = None, shared_gate: Optional[torch.Tensor] = None,
+                 act_dtype: torch.dtype = torch.bfloat16):
+        E = experts_gate_up.num_groups
+        N = E + int(identity)
+        if identity < 0 or router.shape != (N, experts_gate_up.in_features):
+            raise ValueError(f"router weight is {tuple(router.shape)}, expected [{N}, {experts_gate_up.in_features}]")
+        if experts_down.num_groups != E or experts_gate_up.out_features != 2 * experts_down.in_features:
+            raise ValueError("expert gate|up and down weights disagree on the number or width of the experts")
+        if groups < 1 or N % groups or not (1 <= keep <= groups):
+            raise ValueError(f"{N} experts in {groups} groups of which {keep} are kept")
+        if not (1 <= top_k <= min(keep * (N // groups), 32)):
+            raise ValueError(f"experts per row must be 1 .. {min(keep * (N // groups), 32)} here, found {top_k}")
+        if correction is not None and correction.numel() != N:
+            raise ValueError(f"router correction has {correction.numel()} entries for {N} experts")
+        if shared_gate is not None and (shared is None or shared_gate.numel() != router.shape[1]):
+            raise ValueError("a shared expert's gate belongs to a shared expert and has one number per input")
+        self.router, self.correction, self.groups, self.keep = router, correction, int(groups), int(keep)
+        self.experts_gate_up, self.experts_down, self.num_experts, self.identity = experts_gate_up, experts_down, E, int(identity)
+        self.top_k, self.route_scale, self.renormalize, self.limit = int(top_k), float(route_scale), bool(renormalize), float(limit)
+        self.shared, self.shared_gate, self.act_dtype = shared, shared_gate, act_dtype
+        self._tensor_core = (experts_gate_up.weight.dtype == torch.bfloat16
+                             and experts_down.weight.dtype == torch.bfloat16 and act_dtype == torch.bfloat16
+                             and experts_gate_up.in_features % 8 == 0 and experts_down.in_features % 8 == 0)
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, h32: Optional[torch.Tensor] = None,
+                add_to: Optional[torch.Tensor] = None) -> torch.Tensor:
+        T, k, E = h.shape[0], self.top_k, self.num_experts
+        if h32 is None:
+            h32 = h.to(torch.float32)
+        # the shared expert meets the routed ones only in the last sum: it runs on a second stream meanwhile
+        main = torch.cuda.current_stream(h.device)
+        shared = side = None
+        if self.shared is not None:
+            side = _side_stream(h.device)
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                shared = self.shared.forward(ctx, h)
+        expert, weight, gate, _ = ops.router_groups(h32, self.router, k, correction=self.correction, scale=self.route_scale,
+                                                    renormalize=self.renormalize, n_groups=self.groups, keep=self.keep,
+                                                    gate_weight=self.shared_gate)
+        if "router_choices" in ctx.extras:          # tracing: which experts every row went to
+            ctx.extras["router_choices"].append(expert)
+        offsets, sorted_pairs = ops.moe_sort(expert.view(-1), E + self.identity)      # pair = row * k + choice
+        offsets = offsets[: E + 1]                                                    # identity pairs lie behind them
+        pair_rows = ops.moe_pair_tokens(sorted_pairs, k) if k > 1 else sorted_pairs
+        y = torch.empty((T * k, self.experts_down.out_features), dtype=torch.float32, device=h.device)
+        w_pairs = weight.view(-1)
+        if self._tensor_core and h.dtype == torch.bfloat16:
+            h_sorted = ops.gather_rows_bf16(h, pair_rows)
+            w = self.experts_gate_up.weight
+            act = (ops.tc_grouped_gemm_clamped(h_sorted, w, offsets, self.limit) if self.limit > 0
+                   else ops.tc_grouped_gemm(h_sorted, w, offsets, mode=ops.TC_MODE_SWIGLU))
+            ops.tc_grouped_gemm(act, self.experts_down.weight, offsets, mode=ops.TC_MODE_STORE, out=y,
+                                out_rows=sorted_pairs, row_scale=w_pairs, scale_rows=sorted_pairs)
+        else:
+            gu = self.experts_gate_up(h, offsets, rows=T * k, a_rows=pair_rows)        # sorted order
+            w_down = self.experts_down.weight
+            act = torch.empty((T * k, w_down.shape[2]), dtype=self.act_dtype, device=h.device)
+            ops.gated_cols(gu, act, limit=self.limit)
+            if w_down.dtype == torch.float32 and act.dtype != torch.float32:
+                act = act.to(torch.float32)
+            ops.gemm_nt(act, w_down, out=y, group_offsets=offsets, out_rows=sorted_pairs, rows=T * k, row_scale=w_pairs,
+                        scale_rows=sorted_pairs)
+        if side is not None:
+            main.wait_stream(side)
+        return ops.moe_combine_full(y, expert, weight, h32, E, shared=shared, gate=gate, add=add_to, out=add_to)
