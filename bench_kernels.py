@@ -16,6 +16,10 @@
     python bench_kernels.py attention_keys_decode --batch 64 --context 8192     (keys-only pages)
     python bench_kernels.py attention_keys_prefill --tokens 2048 --mask window
     python bench_kernels.py attention_prefill --tokens 2048 --softcap 30 --sinks        (capped scores, sinks)
+    python bench_kernels.py lightning --batch 64 --tokens 1        (linear attention and its gated norm; --batch 1 --tokens 2048)
+    python bench_kernels.py qkv_conv --tokens 2048                 (convolution, rotation, cache write)
+    python bench_kernels.py softmax_mixture --tokens 2048          (router with groups, combine with identity experts)
+    python bench_kernels.py elementwise --op add_rmsnorm_pair --tokens 2048 --hidden 2048
     python bench_kernels.py elementwise --op add_layernorm --tokens 2048 --hidden 2048
 
 Each run warms the kernel up, times ``--iters`` launches with CUDA events and prints one line with
@@ -342,6 +346,15 @@ def elementwise(ns) -> None:
         def fn():
             x, delta = xs()
             ops.add_rmsnorm(x, delta, w, 1e-5, torch.bfloat16, want_fp32=ns.fp32_copy)
+    elif ns.op == "add_rmsnorm_pair":
+        copies = max(2, (300 << 20) // (T * H * 8) + 1)
+        xs = rotate([(torch.randn(T, H, device=DEV), torch.randn(T, H, device=DEV)) for _ in range(copies)])
+        w1, w2 = torch.ones(H, device=DEV), torch.ones(H, device=DEV)
+        nbytes = T * H * (4 + 4 + 4 + 2 + 2 + (4 if ns.fp32_copy else 0))
+
+        def fn():
+            x, delta = xs()
+            ops.add_rmsnorm_pair(x, delta, w1, w2, 1e-5, torch.bfloat16, want_fp32=ns.fp32_copy)
     elif ns.op in ("add_layernorm", "add_dyt"):
         copies = max(2, (300 << 20) // (T * H * 8) + 1)
         xs = rotate([(torch.randn(T, H, device=DEV), torch.randn(T, H, device=DEV)) for _ in range(copies)])
@@ -475,6 +488,110 @@ def ssd(ns) -> None:
           f"(read and written once), {4.0 * T * per_request / ms / 1e9:.2f} TFLOP/s float32")
 
 
+def lightning(ns) -> None:
+    """Linear attention with a constant decay and the norm and gate behind it for `batch` requests of `tokens` rows each:
+    per row and head 4 d dv flops (update of S, S^T q: what the recurrence asks for, whatever form runs it); decode streams
+    the state once."""
+    from sharpinference_b200.parts.lightning import LightningPlanner, lightning_columns
+    B, n, heads, d, dv = ns.batch, ns.tokens, ns.heads, ns.key_dim, ns.value_dim
+    cq, ck, cv, cg, width = lightning_columns(heads, d, dv)
+    T = B * n
+    proj = torch.randn(T, width, device=DEV)
+    powers = ops.decay_powers([1.0 - 2.0 ** (-4 - i % 8) for i in range(heads)]).to(DEV)
+    w = torch.ones(heads * dv, device=DEV)
+    per_request = heads * d * dv
+    copies = max(1, (300 << 20) // (B * per_request * 4) + 1) if n == 1 else 1
+    state = torch.zeros(copies * B, per_request, device=DEV)
+    offs = torch.arange(0, T + 1, n, dtype=torch.int32, device=DEV)
+    slot_sets = [torch.arange(c * B, (c + 1) * B, dtype=torch.int32, device=DEV) for c in range(copies)]
+    planner = LightningPlanner()
+    if ns.walk:
+        planner.WALK_ROWS_UP_TO = 1 << 30
+    plan = planner.plan([0] * B, [n] * B)
+    dev = {k: (torch.from_numpy(v).to(DEV) if v.size else None) for k, v in plan.arrays.items()}
+    out = torch.empty(T, heads * dv, dtype=torch.bfloat16, device=DEV)
+    it = {"i": 0}
+
+    def fn():
+        slots = slot_sets[it["i"] % copies]
+        it["i"] += 1
+        y = ops.lightning(proj, col_q=cq, col_k=ck, col_v=cv, powers=powers, row_offsets=offs, state_slots=slots, state=state,
+                          heads=heads, d=d, dv=dv, num_requests=B, walk_requests=dev["walk"], num_walk=plan.values["num_walk"],
+                          chunks=dev["chunks"], spans=dev["spans"])
+        ops.norm_sigmoid_gate(y, proj[:, cg: cg + heads * dv], w, 1e-6, out)
+    ms = _time(fn, max(ns.iters, copies))
+    print(f"lightning batch={B} tokens={n} heads={heads} d={d} dv={dv}{' walked' if ns.walk else ''}: {ms * 1e3:.1f} us, state "
+          f"{2 * B * per_request * 4 / ms / 1e6:.0f} GB/s (read and written once), {4.0 * T * per_request / ms / 1e9:.2f} TFLOP/s float32")
+
+
+def qkv_conv(ns) -> None:
+    """Short convolution of q, k and v, rotation, q store and cache write for `batch` requests of `tokens` rows each."""
+    from sharpinference_b200.parts.position import leading_rotary_inv_freq_parts
+    B, n, nq, nkv, d, ps = ns.batch, ns.tokens, ns.heads, ns.kv_heads, ns.head_dim, ns.page_size
+    T, C = B * n, (nq + 2 * nkv) * d
+    width = (C + nq + 7) // 8 * 8
+    copies = max(2, (300 << 20) // (T * width * 4) + 1) if T > 64 else 2
+    projs = [torch.randn(T, width, device=DEV) for _ in range(copies)]
+    pages = (n + ps - 1) // ps
+    kv = torch.zeros(B * pages, 2, nkv, ps, d, dtype=torch.bfloat16, device=DEV)
+    table = torch.arange(B * pages, dtype=torch.int32, device=DEV).view(B, pages)
+    positions = torch.arange(n, dtype=torch.int32, device=DEV).repeat(B)
+    row_req = torch.arange(B, dtype=torch.int32, device=DEV).repeat_interleave(n)
+    offs = torch.arange(0, T + 1, n, dtype=torch.int32, device=DEV)
+    slots = torch.arange(B, dtype=torch.int32, device=DEV)
+    state = torch.zeros(B, (ns.taps - 1) * C, device=DEV)
+    w = torch.randn(ns.taps, C, device=DEV)
+    inv, low = (t.to(DEV) for t in leading_rotary_inv_freq_parts(ns.rot, 500000.0))
+    q = torch.empty(T, nq, d, dtype=torch.bfloat16, device=DEV)
+    it = {"i": 0}
+
+    def fn():
+        ops.qkv_conv(projs[it["i"] % copies][:, :C], q, kv, weight=w, state=state, positions=positions, row_req=row_req, row_offsets=offs,
+                     state_slots=slots, block_table=table, nq=nq, nkv=nkv, D=d, key_dim=d, value_dim=d, page_size=ps, inv_freq=inv,
+                     inv_freq_low=low, rot_dims=ns.rot)
+        it["i"] += 1
+    ms = _time(fn, max(ns.iters, copies))
+    print(f"qkv_conv batch={B} tokens={n} heads={nq}/{nkv} d={d} taps={ns.taps}: {ms * 1e3:.1f} us, {T * C * 6 / ms / 1e6:.0f} GB/s")
+
+
+def softmax_mixture(ns) -> None:
+    """The router of a softmax mixture in groups with a gate row, the sum of a row's pairs with identity experts, a gated
+    shared expert and an add-in, and the head gate."""
+    T, H, N, k = ns.tokens, ns.hidden, ns.experts, ns.top
+    copies = max(2, (300 << 20) // (T * H * 4) + 1)
+    hs = [torch.randn(T, H, device=DEV) for _ in range(copies)]
+    wr, corr, gw = torch.randn(N, H, device=DEV) * 0.05, torch.randn(N, device=DEV) * 0.1, torch.randn(H, device=DEV)
+    it = {"i": 0}
+
+    def router():
+        ops.router_groups(hs[it["i"] % copies], wr, k, correction=corr, scale=2.0, n_groups=2, keep=1, gate_weight=gw)
+        it["i"] += 1
+    ms = _time(router, max(ns.iters, copies))
+    print(f"router_groups tokens={T} hidden={H} experts={N} top={k}: {ms * 1e3:.1f} us, {(T * H * 4 + N * H * 4) / ms / 1e6:.0f} GB/s")
+    expert, weight, gate, _ = ops.router_groups(hs[0], wr, k, n_groups=2, keep=1, gate_weight=gw)
+    ys = [torch.randn(T * k, H, device=DEV) for _ in range(2)]
+    shared, add = torch.randn(T, H, device=DEV), torch.randn(T, H, device=DEV)
+
+    def combine():
+        ops.moe_combine_full(ys[it["i"] % 2], expert, weight, hs[it["i"] % copies], N - 2, shared=shared, gate=gate, add=add, out=add)
+        it["i"] += 1
+    ms = _time(combine, max(ns.iters, copies))
+    print(f"moe_combine_full tokens={T} top={k}: {ms * 1e3:.1f} us, {(T * k + 4 * T) * H * 4 / ms / 1e6:.0f} GB/s")
+    heads, D = max(1, H // 128), 128
+    o, g = torch.randn(T, heads, D, device=DEV).to(torch.bfloat16), torch.randn(T, heads, device=DEV)
+    out = torch.empty(T, heads * D, dtype=torch.bfloat16, device=DEV)
+    ms = _time(lambda: ops.gate_heads(o, g, out, heads=heads, D=D, dv=D), max(ns.iters, 8))
+    print(f"gate_heads tokens={T} heads={heads}: {ms * 1e3:.1f} us, {T * heads * D * 4 / ms / 1e6:.0f} GB/s")
+    gu = [torch.randn(T, 8 * H, device=DEV) for _ in range(2)]
+    bias, wide = torch.randn(8 * H, device=DEV), torch.empty(T, 4 * H + 8, dtype=torch.bfloat16, device=DEV)
+
+    def gated():
+        ops.gated_cols(gu[it["i"] % 2], wide, bias=bias, ones=3)
+        it["i"] += 1
+    ms = _time(gated, max(ns.iters, 8))
+    print(f"gated_cols tokens={T} ff={4 * H}: {ms * 1e3:.1f} us, {T * 4 * H * 10 / ms / 1e6:.0f} GB/s")
+
+
 def _keys_cache(batch: int, context: int, nkv: int, d: int, ps: int):
     blocks = (context + ps - 1) // ps
     pages = batch * blocks
@@ -553,7 +670,7 @@ def main(argv=None) -> int:
     p.add_argument("--impl", choices=["grouped", "rows", "library"], default="grouped")
     p.set_defaults(fn=dense)
     p = sub.add_parser("elementwise")
-    p.add_argument("--op", choices=["add_rmsnorm", "swiglu", "gather", "qkv_post", "add_layernorm", "add_dyt", "qkv_post_wide"], default="add_rmsnorm")
+    p.add_argument("--op", choices=["add_rmsnorm", "add_rmsnorm_pair", "swiglu", "gather", "qkv_post", "add_layernorm", "add_dyt", "qkv_post_wide"], default="add_rmsnorm")
     p.add_argument("--tokens", type=int, default=2048)
     p.add_argument("--hidden", type=int, default=5120)
     p.add_argument("--inter", type=int, default=8192)
@@ -643,6 +760,30 @@ def main(argv=None) -> int:
         p.add_argument("--keep-first", type=int, default=0)
         p.add_argument("--bias-far", type=int, default=0, help="rows of a distance-bias table minus one (0: no bias)")
         p.set_defaults(fn=fn)
+    p = sub.add_parser("lightning")
+    p.add_argument("--batch", type=int, default=64)
+    p.add_argument("--tokens", type=int, default=1)
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--key-dim", type=int, default=128)
+    p.add_argument("--value-dim", type=int, default=128)
+    p.add_argument("--walk", action="store_true", help="walk the rows one by one whatever their number")
+    p.set_defaults(fn=lightning)
+    p = sub.add_parser("qkv_conv")
+    p.add_argument("--batch", type=int, default=1)
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--kv-heads", type=int, default=4)
+    p.add_argument("--head-dim", type=int, default=128)
+    p.add_argument("--page-size", type=int, default=64)
+    p.add_argument("--taps", type=int, default=4)
+    p.add_argument("--rot", type=int, default=64)
+    p.set_defaults(fn=qkv_conv)
+    p = sub.add_parser("softmax_mixture")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--hidden", type=int, default=2048)
+    p.add_argument("--experts", type=int, default=18)
+    p.add_argument("--top", type=int, default=2)
+    p.set_defaults(fn=softmax_mixture)
     for sp in sub.choices.values():
         sp.add_argument("--iters", type=int, default=10)
         sp.add_argument("--graph", action="store_true", help="time replays of a CUDA graph of the calls")

@@ -765,10 +765,42 @@ gate_heads_kernel(const TO* o, const float* g, int ld_g, TO* out, int ld_out, in
     }
 }
 
+// the same eight elements a thread (16-byte accesses for 16-bit heads), sizes and places that are multiples of eight
+template <typename TO>
+__global__ void __launch_bounds__(256)
+gate_heads_vec8_kernel(const TO* o, const float* g, int ld_g, TO* out, int ld_out, int heads, int D, int dv, float scale,
+                       long long n) {
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const int per = dv / 8;
+    const long long th = i / per;
+    const int e = (int)(i - th * per) * 8;
+    const int t = (int)(th / heads), h = (int)(th - (long long)t * heads);
+    const float f = scale / (1.0f + expf(-g[(size_t)t * ld_g + h]));
+    struct alignas(16) Eight { TO v[8]; };
+    Eight x = *reinterpret_cast<const Eight*>(o + (size_t)th * D + e);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x.v[j] = from_float<TO>(to_float(x.v[j]) * f);
+    *reinterpret_cast<Eight*>(out + (size_t)t * ld_out + (size_t)h * dv + e) = x;
+}
+
 SHARPI_API int sharpi_gate_heads(const void* o, const float* g, int ld_g, void* out, int ld_out, int dtype, int T, int heads,
                                  int D, int dv, float scale, cudaStream_t stream) {
     if (T <= 0) return SHARPI_OK;
     if (heads <= 0 || dv <= 0 || D < dv || ld_g < heads || ld_out < heads * dv) return SHARPI_BAD_ARGUMENT;
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(out);
+    if (D % 8 == 0 && dv % 8 == 0 && ld_out % 8 == 0 && (ptrs & 15) == 0) {
+        const long long n = (long long)T * heads * (dv / 8);
+        const unsigned blocks = (unsigned)((n + 255) / 256);
+        if (dtype == SHARPI_F32)
+            SHARPI_LAUNCH_PDL(gate_heads_vec8_kernel<float>, blocks, 256, 0, stream, (const float*)o, g, ld_g, (float*)out, ld_out, heads, D, dv, scale, n);
+        else if (dtype == SHARPI_BF16)
+            SHARPI_LAUNCH_PDL(gate_heads_vec8_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)o, g, ld_g, (bf16*)out, ld_out, heads, D, dv, scale, n);
+        else
+            return SHARPI_BAD_ARGUMENT;
+        return SHARPI_OK;
+    }
     int by = (heads * dv + 1023) / 1024;
     const dim3 grid(T, by > 64 ? 64 : by);
     if (dtype == SHARPI_F32)

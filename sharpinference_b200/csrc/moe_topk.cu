@@ -21,57 +21,69 @@
 // routing stays on the device so that a step's rows can be sorted by expert for grouped products.
 #include "common.cuh"
 
-constexpr int TOPK_WARPS = 8;
 constexpr int TOPK_MANY_ROWS = 512;   // steps of more rows than this put four rows in a CTA (a router row is fetched
                                       // once for all of them); smaller steps one, for more CTAs
 
-// One CTA per TOPK_ROWS rows (1 or 4): warp w forms the logits of experts w, w + 8, ... for each of the CTA's rows (a lane
-// adds its elements of a row in ascending order in four interleaved chains, the chains and then the lanes are added
-// in a fixed order: a row's logits do not depend on its neighbours), then warp r picks the k best of row r.
+// One CTA per TOPK_ROWS rows (1 or 4): warp w forms the logits of experts w, w + warps, ... for each of the CTA's rows: lane
+// l adds the elements 128 i + 4 l + u in ascending i into chain u = 0 .. 3, the chains and then the lanes are added in a
+// fixed order, so a row's logits depend on neither its neighbours nor the number of warps.  Then warp r picks the k best of
+// row r.
 template <int TOPK_ROWS>
-__global__ void __launch_bounds__(TOPK_WARPS * 32)
+__global__ void __launch_bounds__(1024)
 router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                    int T, int H, int E, int k, float scale, int renormalize, int* __restrict__ expert_id,
                    float* __restrict__ weight, float* __restrict__ scores_out, int stage_rows,
                    const float* __restrict__ bias, int scoring, int n_groups, int keep, const float* __restrict__ gate_w,
-                   float* __restrict__ gate_out) {
-    extern __shared__ float smem[];                       // per row s [E], choice [E]; group scores; then the rows [ROWS][H] if they fit
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+                   float* __restrict__ gate_out, int vec) {
+    extern __shared__ __align__(16) float smem[];         // the rows [ROWS][H] if they fit; per row s [E], choice [E]; group scores
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int t0 = blockIdx.x * TOPK_ROWS;
     const int rows = min(TOPK_ROWS, T - t0);
+    float* const score_s = smem + (stage_rows ? ((size_t)TOPK_ROWS * H + 3) / 4 * 4 : 0);
     const float* row[TOPK_ROWS];
 #pragma unroll
     for (int r = 0; r < TOPK_ROWS; ++r) row[r] = h + (size_t)(t0 + min(r, rows - 1)) * H;
     if (stage_rows) {                                     // the rows are read from memory once, by all warps together
-        float* rows_s = smem + (size_t)TOPK_ROWS * (2 * E + n_groups);
-        for (int i = threadIdx.x; i < rows * H; i += TOPK_WARPS * 32) rows_s[i] = h[(size_t)t0 * H + i];
+        if (vec) {
+            const float4* src = reinterpret_cast<const float4*>(h + (size_t)t0 * H);
+            for (int i = threadIdx.x; i < rows * H / 4; i += blockDim.x) reinterpret_cast<float4*>(smem)[i] = src[i];
+        } else {
+            for (int i = threadIdx.x; i < rows * H; i += blockDim.x) smem[i] = h[(size_t)t0 * H + i];
+        }
         __syncthreads();
 #pragma unroll
-        for (int r = 0; r < TOPK_ROWS; ++r) row[r] = rows_s + (size_t)min(r, rows - 1) * H;
+        for (int r = 0; r < TOPK_ROWS; ++r) row[r] = smem + (size_t)min(r, rows - 1) * H;
     }
-    for (int e = warp; e < E + (gate_w ? 1 : 0); e += TOPK_WARPS) {
+    for (int e = warp; e < E + (gate_w ? 1 : 0); e += warps) {
         const float* w = e < E ? wr + (size_t)e * H : gate_w;
         float acc[TOPK_ROWS][4];
 #pragma unroll
         for (int r = 0; r < TOPK_ROWS; ++r)
 #pragma unroll
             for (int u = 0; u < 4; ++u) acc[r][u] = 0.0f;
-        int i = lane;
-        for (; i + 96 < H; i += 128) {
+        if (vec) {
+#pragma unroll 4
+            for (int i = 4 * lane; i < H; i += 128) {
+                const float4 wv = *reinterpret_cast<const float4*>(w + i);
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const float wv = w[i + 32 * u];
-#pragma unroll
-                for (int r = 0; r < TOPK_ROWS; ++r) acc[r][u] = fmaf(row[r][i + 32 * u], wv, acc[r][u]);
+                for (int r = 0; r < TOPK_ROWS; ++r) {
+                    const float4 x = *reinterpret_cast<const float4*>(row[r] + i);
+                    acc[r][0] = fmaf(x.x, wv.x, acc[r][0]);
+                    acc[r][1] = fmaf(x.y, wv.y, acc[r][1]);
+                    acc[r][2] = fmaf(x.z, wv.z, acc[r][2]);
+                    acc[r][3] = fmaf(x.w, wv.w, acc[r][3]);
+                }
             }
-        }
+        } else {
+            for (int i = 4 * lane; i < H; i += 128) {
 #pragma unroll
-        for (int u = 0; u < 3; ++u) {                      // what is left: up to three more elements a lane
-            const int ii = i + 32 * u;
-            if (ii < H) {
-                const float wv = w[ii];
+                for (int u = 0; u < 4; ++u) {
+                    if (i + u < H) {
+                        const float wv = w[i + u];
 #pragma unroll
-                for (int r = 0; r < TOPK_ROWS; ++r) acc[r][u] = fmaf(row[r][ii], wv, acc[r][u]);
+                        for (int r = 0; r < TOPK_ROWS; ++r) acc[r][u] = fmaf(row[r][i + u], wv, acc[r][u]);
+                    }
+                }
             }
         }
 #pragma unroll
@@ -80,8 +92,8 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
             if (lane == 0 && r < rows && e == E) gate_out[t0 + r] = 1.0f / (1.0f + expf(-z));
             if (lane == 0 && r < rows && e < E) {
                 const float s = scoring >= 1 ? z : 1.0f / (1.0f + expf(-z));
-                smem[(size_t)r * 2 * E + e] = s;
-                smem[(size_t)r * 2 * E + E + e] = correction ? s + correction[e] : s;
+                score_s[(size_t)r * 2 * E + e] = s;
+                score_s[(size_t)r * 2 * E + E + e] = correction ? s + correction[e] : s;
                 if (scores_out && scoring != 2) scores_out[(size_t)(t0 + r) * E + e] = s;
             }
         }
@@ -89,7 +101,7 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
     __syncthreads();
     if (warp >= rows) return;
     const int t = t0 + warp;
-    float* s_s = smem + (size_t)warp * 2 * E;
+    float* s_s = score_s + (size_t)warp * 2 * E;
     float* c_s = s_s + E;
     if (scoring == 2) {
         float m = -INFINITY, sum = 0.0f;
@@ -109,7 +121,7 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
         }
         __syncwarp();
         if (n_groups > 1 && keep < n_groups) {
-            float* g_s = smem + (size_t)TOPK_ROWS * 2 * E + (size_t)warp * n_groups;       // a group's largest choice score
+            float* g_s = score_s + (size_t)TOPK_ROWS * 2 * E + (size_t)warp * n_groups;       // a group's largest choice score
             const int per = E / n_groups;
             for (int g = lane; g < n_groups; g += 32) {
                 float best = -INFINITY;
@@ -173,16 +185,22 @@ static int router_topk_impl(const float* h, const float* wr, const float* correc
     const int per_cta = T > TOPK_MANY_ROWS ? 4 : 1;
     size_t smem = (size_t)per_cta * (2 * E + n_groups) * sizeof(float);
     if (smem > 48 * 1024) return SHARPI_BAD_ARGUMENT;
-    const int stage_rows = smem + (size_t)per_cta * H * sizeof(float) <= 48 * 1024;
-    if (stage_rows) smem += (size_t)per_cta * H * sizeof(float);
+    const size_t copies = ((size_t)per_cta * H + 3) / 4 * 4 * sizeof(float);
+    const int stage_rows = smem + copies <= 48 * 1024;
+    if (stage_rows) smem += copies;
+    const int vec = H % 4 == 0 && ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(wr) |
+                                    reinterpret_cast<uintptr_t>(gate_w)) & 15) == 0;
+    // a warp an expert where the step is small (the wait is what counts), eight where its CTAs fill the GPU
+    const int experts = E + (gate_w ? 1 : 0);
+    const int warps = T > TOPK_MANY_ROWS ? 8 : experts < 8 ? 8 : experts > 32 ? 32 : experts;
     if (per_cta == 4)
-        router_topk_kernel<4><<<(T + 3) / 4, TOPK_WARPS * 32, smem, stream>>>(
+        router_topk_kernel<4><<<(T + 3) / 4, warps * 32, smem, stream>>>(
             h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring,
-            n_groups, keep, gate_w, gate_out);
+            n_groups, keep, gate_w, gate_out, vec);
     else
-        router_topk_kernel<1><<<T, TOPK_WARPS * 32, smem, stream>>>(
+        router_topk_kernel<1><<<T, warps * 32, smem, stream>>>(
             h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring,
-            n_groups, keep, gate_w, gate_out);
+            n_groups, keep, gate_w, gate_out, vec);
     SHARPI_CHECK_LAUNCH();
     return SHARPI_OK;
 }

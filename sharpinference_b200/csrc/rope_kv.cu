@@ -649,6 +649,7 @@ struct QkvConvArgs {
     const int* state_slots;
     const int* block_table;
     const float* inv_freq;   // [rot / 2] or null
+    const float* inv_low;    // [rot / 2] or null: what the float32 frequencies leave of the exact ones
     void* q_out;             // [T, nq, D]
     void* kv_base;           // [page][2][nkv][page_size][D]
     int T, nq, nkv, D, dk, dv, rot, pairing;
@@ -666,6 +667,18 @@ template <int VEC> __device__ __forceinline__ void read_vec(const float* p, floa
 template <typename TO, int VEC> __device__ __forceinline__ void write_vec(TO* p, const float* v) {
     if (VEC == 4) store4<TO>(p, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
     else *p = from_float<TO>(v[0]);
+}
+
+// Sine and cosine of pos * f.  The product is rounded to float32 (half a unit of a large angle is a visible turn), so what
+// that rounding and the frequency's own float32 form leave out, a small angle, is turned on behind it.
+__device__ __forceinline__ void conv_turn(const QkvConvArgs& a, int pair, float pos, float* sn, float* cs) {
+    const float f = a.inv_freq[pair], angle = pos * f;
+    const float rest = fmaf(pos, f, -angle) + (a.inv_low ? pos * a.inv_low[pair] : 0.0f);
+    float s0, c0;
+    sincosf(angle, &s0, &c0);
+    const float one = 1.0f - 0.5f * rest * rest;
+    *sn = fmaf(c0, rest, s0 * one);
+    *cs = fmaf(-s0, rest, c0 * one);
 }
 
 template <typename TO, int VEC>
@@ -738,7 +751,7 @@ __global__ void __launch_bounds__(256) qkv_conv_kernel(QkvConvArgs a) {
 #pragma unroll
                 for (int u = 0; u < VEC; ++u) {
                     float sn, cs;
-                    sincosf((float)pos * a.inv_freq[e + u], &sn, &cs);
+                    conv_turn(a, e + u, (float)pos, &sn, &cs);
                     const float y0 = y[u] * cs - z[u] * sn, z0 = z[u] * cs + y[u] * sn;
                     y[u] = y0;
                     z[u] = z0;
@@ -757,10 +770,154 @@ __global__ void __launch_bounds__(256) qkv_conv_kernel(QkvConvArgs a) {
         }
 }
 
+// The form for heads of up to 128 elements whose sizes and places are multiples of four: a lane owns four neighbouring
+// channels of a head, a warp walks R rows of the step with the last TAPS inputs in registers (an input is fetched once for
+// all the outputs it enters, and all R rows are asked for at once), the partner of a rotated element comes from another
+// lane, and the block's sines and cosines are formed once for its eight heads.  The additions are those of the kernel above.
+// Rows of a portion whose window reaches before the portion's start are served by the warp of its first row, also where they
+// lie behind that warp's R rows.
+template <typename TO, int TAPS, int R>
+__global__ void __launch_bounds__(256) qkv_conv_rows_kernel(QkvConvArgs a) {
+    constexpr int ROWS = R + TAPS - 2;                         // rows a warp may serve: its own, and up to TAPS - 2 behind
+    __shared__ __align__(16) float sn_s[ROWS][64];
+    __shared__ __align__(16) float cs_s[ROWS][64];
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * R;
+    const int half = a.rot >> 1;
+    if (half > 0) {
+        for (int i = threadIdx.x; i < ROWS * half; i += blockDim.x) {
+            const int r = i / half, j = i - r * half;
+            if (t0 + r < a.T) conv_turn(a, j, (float)a.positions[t0 + r], &sn_s[r][j], &cs_s[r][j]);
+        }
+        __syncthreads();
+    }
+    const int slots = a.nq + 2 * a.nkv;
+    const int slot = blockIdx.y * 8 + warp;
+    if (slot >= slots) return;
+    const bool is_q = slot < a.nq;
+    const bool is_v = slot >= a.nq + a.nkv;
+    const int size = is_v ? a.dv : a.dk;
+    const int ch0 = is_v ? (a.nq + a.nkv) * a.dk + (slot - a.nq - a.nkv) * a.dv : slot * a.dk;
+    const int head = is_v ? slot - a.nq - a.nkv : slot - a.nq;
+    const int e = lane * 4;
+    const bool own = e < size, inside = e < a.D;
+    const int keep = a.taps - 1;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const float* in = a.proj + a.col0 + ch0 + e;
+    // where the lane's partner sits: first halves meet the lanes half / 4 above, second halves those below
+    const bool turned = !is_v && e < a.rot, low = e < half;
+    const int partner = turned ? (low ? lane + half / 4 : lane - half / 4) : lane;
+    const int pair = low ? e : e - half;
+    float4 w[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+        const int tap = j - (TAPS - a.taps);                   // the last tap sits in the last place
+        w[j] = own && tap >= 0 ? *reinterpret_cast<const float4*>(a.w + (size_t)tap * a.C + ch0 + e) : zero;
+    }
+    float4 pre[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+        pre[r] = own && t0 + r < a.T ? *reinterpret_cast<const float4*>(in + (size_t)(t0 + r) * a.ld) : zero;
+    float4 win[TAPS];
+    int cur = -1, first = 0, n = 0;
+    bool lead = false;
+    float* st = nullptr;
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int t = t0 + r;
+        if (t >= a.T) break;
+        if (r >= R && !(lead && t - first < min(keep, n))) break;
+        const int b = a.row_req[t];
+        if (b != cur) {                                        // a portion begins, or the warp's rows begin inside one
+            if (r >= R) break;
+            cur = b;
+            first = a.row_offsets[b];
+            n = a.row_offsets[b + 1] - first;
+            lead = t == first;
+            if (keep > 0) st = a.state + (size_t)a.state_slots[b] * a.state_stride + ch0 + e;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {                   // the window before this row: win[TAPS - back] for back inputs ago
+                win[j] = zero;
+                const int back = TAPS - j;
+                if (own && back <= keep) {
+                    const int at = t - first - back;
+                    if (at >= 0) win[j] = *reinterpret_cast<const float4*>(in + (size_t)(t - back) * a.ld);
+                    else if (lead) win[j] = *reinterpret_cast<const float4*>(st + (size_t)(keep + at) * a.C);
+                }
+            }
+        }
+        const int i = t - first;
+        const float4 x = r < R ? pre[r < R ? r : 0] : (own ? *reinterpret_cast<const float4*>(in + (size_t)t * a.ld) : zero);
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
+        win[TAPS - 1] = x;
+        if (i < keep && !lead) continue;                       // the portion's first row serves this one
+        float4 y = zero;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            y.x = fmaf(w[j].x, win[j].x, y.x);
+            y.y = fmaf(w[j].y, win[j].y, y.y);
+            y.z = fmaf(w[j].z, win[j].z, y.z);
+            y.w = fmaf(w[j].w, win[j].w, y.w);
+        }
+        if (half > 0 && !is_v) {
+            float4 o;
+            o.x = __shfl_sync(0xffffffffu, y.x, partner);
+            o.y = __shfl_sync(0xffffffffu, y.y, partner);
+            o.z = __shfl_sync(0xffffffffu, y.z, partner);
+            o.w = __shfl_sync(0xffffffffu, y.w, partner);
+            if (turned) {
+                float4 sn = *reinterpret_cast<const float4*>(&sn_s[r][pair]);
+                const float4 cs = *reinterpret_cast<const float4*>(&cs_s[r][pair]);
+                if (low) { sn.x = -sn.x; sn.y = -sn.y; sn.z = -sn.z; sn.w = -sn.w; }
+                y.x = y.x * cs.x + o.x * sn.x;
+                y.y = y.y * cs.y + o.y * sn.y;
+                y.z = y.z * cs.z + o.z * sn.z;
+                y.w = y.w * cs.w + o.w * sn.w;
+            }
+        }
+        if (inside) {
+            if (is_q) {
+                store4<TO>((TO*)a.q_out + ((size_t)t * a.nq + slot) * a.D + e, y);
+            } else {
+                const int pos = a.positions[t];
+                const int page = a.block_table[(size_t)b * a.max_blocks + pos / a.page_size];
+                if (page >= 0)                                 // the host checks that written positions have pages
+                    store4<TO>((TO*)a.kv_base + (((size_t)page * 2 + (is_v ? 1 : 0)) * a.nkv + head) * a.page_size * a.D +
+                                   (size_t)(pos % a.page_size) * a.D + e, y);
+            }
+        }
+        if (lead && own && keep > 0 && i == min(keep, n) - 1) {    // the rows that read the old state are served: move it on
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                const int at = j - (TAPS - keep);              // place in the state
+                if (at < 0) continue;
+                const float4 v = n <= keep ? win[j] : *reinterpret_cast<const float4*>(in + (size_t)(first + n - keep + at) * a.ld);
+                *reinterpret_cast<float4*>(st + (size_t)at * a.C) = v;
+            }
+        }
+    }
+}
+
+template <typename TO, int TAPS>
+static int launch_conv_rows(const QkvConvArgs& a, cudaStream_t stream) {
+    const int groups = (a.nq + 2 * a.nkv + 7) / 8;
+    if (a.T <= 256) {                                          // few rows: a warp each, for the shortest wait
+        auto kern = qkv_conv_rows_kernel<TO, TAPS, 1>;
+        SHARPI_LAUNCH_PDL(kern, dim3(a.T, groups), 256, 0, stream, a);
+    } else {
+        auto kern = qkv_conv_rows_kernel<TO, TAPS, 8>;
+        SHARPI_LAUNCH_PDL(kern, dim3((a.T + 7) / 8, groups), 256, 0, stream, a);
+    }
+    return SHARPI_OK;
+}
+
 SHARPI_API int sharpi_qkv_conv(const float* proj, int ld, int col0, const float* w, int taps, float* state,
                                long long state_stride, const int* positions, const int* row_req, const int* row_offsets,
-                               const int* state_slots, const int* block_table, const float* inv_freq, int rot, int pairing,
-                               void* q_out, void* kv_base, int out_dtype, int T, int nq, int nkv, int D, int dk, int dv,
+                               const int* state_slots, const int* block_table, const float* inv_freq, const float* inv_low,
+                               int rot, int pairing, void* q_out, void* kv_base, int out_dtype, int T, int nq, int nkv, int D,
+                               int dk, int dv,
                                int max_blocks, int page_size, cudaStream_t stream) {
     if (T <= 0) return SHARPI_OK;
     if (nq <= 0 || nkv <= 0 || D <= 0 || dk <= 0 || dk > D || dv <= 0 || dv > D || page_size <= 0 || max_blocks <= 0 ||
@@ -773,13 +930,18 @@ SHARPI_API int sharpi_qkv_conv(const float* proj, int ld, int col0, const float*
     if (col0 < 0 || col0 + a.C > ld) return SHARPI_BAD_ARGUMENT;
     a.proj = proj; a.ld = ld; a.col0 = col0; a.w = w; a.taps = taps; a.state = state; a.state_stride = state_stride;
     a.positions = positions; a.row_req = row_req; a.row_offsets = row_offsets; a.state_slots = state_slots;
-    a.block_table = block_table; a.inv_freq = inv_freq; a.q_out = q_out; a.kv_base = kv_base;
+    a.block_table = block_table; a.inv_freq = inv_freq; a.inv_low = inv_low; a.q_out = q_out; a.kv_base = kv_base;
     a.T = T; a.nq = nq; a.nkv = nkv; a.D = D; a.dk = dk; a.dv = dv; a.rot = rot; a.pairing = pairing;
     a.max_blocks = max_blocks; a.page_size = page_size;
     const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(state) |
                            reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(kv_base);
     const bool vec = dk % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && (rot / 2) % 4 == 0 &&
                      (rot == 0 || pairing == ROPE_HALVES) && state_stride % 4 == 0 && (ptrs & 15) == 0;
+    if (vec && D <= 128 && taps <= 8) {                        // (half a rotation is then a multiple of four: see vec)
+        if (out_dtype == SHARPI_F32) return taps <= 4 ? launch_conv_rows<float, 4>(a, stream) : launch_conv_rows<float, 8>(a, stream);
+        if (out_dtype == SHARPI_BF16) return taps <= 4 ? launch_conv_rows<bf16, 4>(a, stream) : launch_conv_rows<bf16, 8>(a, stream);
+        return SHARPI_BAD_ARGUMENT;
+    }
     const long long work = (long long)T * (nq + 2 * nkv);
     const long long blocks = (work + 7) / 8;
     if (blocks > 2147483647LL) return SHARPI_BAD_ARGUMENT;

@@ -1572,10 +1572,12 @@ def softcap_(y: torch.Tensor, cap: float) -> torch.Tensor:
 def qkv_conv(proj: torch.Tensor, q_out: torch.Tensor, kv_layer: torch.Tensor, *, weight: torch.Tensor,
              state: Optional[torch.Tensor], positions: torch.Tensor, row_req: torch.Tensor, row_offsets: torch.Tensor,
              state_slots: torch.Tensor, block_table: torch.Tensor, nq: int, nkv: int, D: int, key_dim: int, value_dim: int,
-             page_size: int, inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0, pairing: int = ROPE_HALVES) -> None:
+             page_size: int, inv_freq: Optional[torch.Tensor] = None, inv_freq_low: Optional[torch.Tensor] = None,
+             rot_dims: int = 0, pairing: int = ROPE_HALVES) -> None:
     """Causal convolution of every channel of q | k | v (``proj`` float32 ``[T, C]``, a column range of a wider product, heads
     unpadded), rotation of the first ``rot_dims`` elements of q and k, q store (``q_out`` ``[T, nq, D]``, zeros behind
-    ``key_dim``) and the scatter of k and v into pages.  ``weight`` float32 ``[taps, C]``; ``state`` float32
+    ``key_dim``) and the scatter of k and v into pages.  ``inv_freq_low``: what the float32 frequencies leave of the exact
+    ones (:func:`parts.position.leading_rotary_inv_freq_parts`).  ``weight`` float32 ``[taps, C]``; ``state`` float32
     ``[slots, (taps - 1) * C]``, read and moved on."""
     ld = _need_columns(proj, "proj", torch.float32)
     _need(weight, "weight", torch.float32)
@@ -1598,11 +1600,15 @@ def qkv_conv(proj: torch.Tensor, q_out: torch.Tensor, kv_layer: torch.Tensor, *,
         _need(inv_freq, "inv_freq", torch.float32)
         if inv_freq.numel() != rot_dims // 2:
             raise KernelError(f"{rot_dims} rotated elements need {rot_dims // 2} frequencies, found {inv_freq.numel()}")
+        if inv_freq_low is not None:
+            _need(inv_freq_low, "inv_freq_low", torch.float32)
+            if inv_freq_low.numel() != rot_dims // 2:
+                raise KernelError(f"inv_freq_low has {inv_freq_low.numel()} entries, expected {rot_dims // 2}")
     check(kernel("sharpi_qkv_conv")(proj.data_ptr(), ld, 0, weight.data_ptr(), taps, _ptr(state) if taps > 1 else None,
                                     state.stride(0) if taps > 1 else 0, positions.data_ptr(), row_req.data_ptr(),
                                     row_offsets.data_ptr(), state_slots.data_ptr(), block_table.data_ptr(),
-                                    _ptr(inv_freq) if rot_dims else None, int(rot_dims), int(pairing), q_out.data_ptr(),
-                                    kv_layer.data_ptr(), dtype_code(q_out.dtype), T, nq, nkv, D, key_dim, value_dim,
+                                    _ptr(inv_freq) if rot_dims else None, _ptr(inv_freq_low) if rot_dims else None,
+                                    int(rot_dims), int(pairing), q_out.data_ptr(), kv_layer.data_ptr(), dtype_code(q_out.dtype), T, nq, nkv, D, key_dim, value_dim,
                                     block_table.shape[-1], page_size, _stream()), "sharpi_qkv_conv")
 
 

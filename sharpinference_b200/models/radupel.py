@@ -25,7 +25,7 @@ import torch
 from ..config.radupel import RadupelConfig, RadupelLayer
 from ..parts import (AddInput, ConvAttention, DenseSwiGLU, GroupedLinear, LightningAttention, Linear, MoESoftmaxGroups,
                      ParallelPairBlock, RMSNorm, RotaryEncoding, ScaledBranches, conv_attention_columns,
-                     leading_rotary_inv_freq, lightning_columns)
+                     leading_rotary_inv_freq_parts, lightning_columns)
 from ..registry import register_architecture
 from ..weights.source import WeightSource
 from .model import DecoderModel, ScheduleEntry
@@ -53,9 +53,10 @@ def _attention(c: RadupelConfig, layer: RadupelLayer, p: str, weights: WeightSou
     out = weights.matrix(p + "o", (W, H * dv))
     position = None
     if a.rot_dims:
-        inv_freq = leading_rotary_inv_freq(a.rot_dims, a.rot_base)
-        position = RotaryEncoding(inv_freq if weights.device.type == "meta" else inv_freq.to(weights.device), "halves",
-                                  a.rot_dims)
+        high, low = leading_rotary_inv_freq_parts(a.rot_dims, a.rot_base)
+        if weights.device.type != "meta":
+            high, low = high.to(weights.device), low.to(weights.device)
+        position = RotaryEncoding(high, "halves", a.rot_dims, inv_freq_low=low)
     return ConvAttention(proj=_padded(rows, conv_attention_columns(H, G, d, dv)[1]), out=out,
                          conv_weight=taps.t().contiguous(), num_heads=H, num_kv_heads=G, key_dim=d, value_dim=dv,
                          softmax_scale=a.scale, position=position, act_dtype=act, name=p)

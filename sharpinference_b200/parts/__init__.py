@@ -3,8 +3,8 @@ from .base import (Block, CacheSpec, ColumnMixer, FeedForward, LayerSlot, Mixer,
                    StepContext, StreamOp, make_part, part_kinds, register_part)
 from .linear import GroupedLinear, Linear
 from .norm import DynamicTanh, L2Norm, LayerNorm, RMSNorm
-from .position import (NoPositionEncoding, RotaryEncoding, leading_rotary_inv_freq, partial_rotary_inv_freq,
-                       rotary_inv_freq, yarn_inv_freq)
+from .position import (NoPositionEncoding, RotaryEncoding, leading_rotary_inv_freq, leading_rotary_inv_freq_parts,
+                       partial_rotary_inv_freq, rotary_inv_freq, yarn_inv_freq)
 from .attention import PagedAttention, distance_bias_table, distance_bucket
 from .latent import LatentAttention
 from .mlstm import MLSTMMixer, fused_mlstm_columns
@@ -26,4 +26,4 @@ __all__ = ["Block", "CacheSpec", "FeedForward", "LayerSlot", "Mixer", "Norm", "P
            "HyperBlock", "PairEmbedding", "WKVMixer", "BranchPair", "SelectiveScanMixer", "leading_rotary_inv_freq", "DynamicTanh", "LatentAttention", "MoESigmoidTopKGated", "StateSpaceDualityMixer",
            "ssd_projection_order", "distance_bias_table", "distance_bucket", "LayerNorm", "yarn_inv_freq",
            "ColumnMixer", "ConvAttention", "conv_attention_columns", "LightningAttention", "LightningPlanner", "lightning_columns",
-           "ScaledBranches", "ParallelPairBlock", "AddInput", "MoESoftmaxGroups"]
+           "ScaledBranches", "ParallelPairBlock", "AddInput", "MoESoftmaxGroups", "leading_rotary_inv_freq_parts"]

@@ -16,6 +16,7 @@ import torch
 from .base import ColumnMixer, LayerSlot, StepContext, StepPlanner, register_part
 from .linear import Linear
 from .mamba import BranchPair
+from .side import fork
 
 
 def pad_columns(n: int) -> int:
@@ -59,13 +60,18 @@ class ScaledBranches(ColumnMixer):
     def step_planners(self, page_size: int) -> List[StepPlanner]:
         return self.left.step_planners(page_size) + self.right.step_planners(page_size)
 
+    def _branch(self, ctx, slot, m: ColumnMixer, prefix: str, proj, out, at: int, col: int, scale: float) -> None:
+        m.inner(ctx, BranchPair._branch_slot(slot, prefix, m), proj[:, at: at + m.in_columns],
+                out[:, col: col + m.out_columns], scale=scale)
+        gap = pad_columns(m.out_columns) - m.out_columns
+        if gap:                                            # the output weight has zero columns there: no NaN may stand in them
+            out[:, col + m.out_columns: col + m.out_columns + gap].zero_()
+
     def inner(self, ctx: StepContext, slot: LayerSlot, proj: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-        at = 0
-        for m, prefix, factor, col in ((self.left, "left.", self.left_scale, 0),
-                                       (self.right, "right.", self.right_scale, self._right_at)):
-            m.inner(ctx, BranchPair._branch_slot(slot, prefix, m), proj[:, at: at + m.in_columns],
-                    out[:, col: col + m.out_columns], scale=scale * factor)
-            gap = pad_columns(m.out_columns) - m.out_columns
-            if gap:                                        # the output weight has zero columns there: no NaN may stand in them
-                out[:, col + m.out_columns: col + m.out_columns + gap].zero_()
-            at += m.in_columns
+        # the branches meet in the output product: the right one runs on a stream of its own
+        side = fork(proj.device, "branch")
+        with torch.cuda.stream(side):
+            self._branch(ctx, slot, self.right, "right.", proj, out, self.left.in_columns, self._right_at,
+                         scale * self.right_scale)
+        self._branch(ctx, slot, self.left, "left.", proj, out, 0, 0, scale * self.left_scale)
+        torch.cuda.current_stream(proj.device).wait_stream(side)

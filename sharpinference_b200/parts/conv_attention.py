@@ -47,7 +47,7 @@ class ConvAttention(ColumnMixer, PagedAttention):
                              f"{num_heads * value_dim}")
         if conv_weight.dim() != 2 or conv_weight.shape[1] != channels or conv_weight.shape[0] < 1:
             raise ValueError(f"the convolution is {tuple(conv_weight.shape)}, expected [taps, {channels}]")
-        self.rot_dims, self.inv_freq, self.pairing = 0, None, ops.ROPE_HALVES
+        self.rot_dims, self.inv_freq, self.inv_freq_low, self.pairing = 0, None, None, ops.ROPE_HALVES
         if position is not None:
             rot = position.rotary()
             if rot is None:
@@ -55,6 +55,7 @@ class ConvAttention(ColumnMixer, PagedAttention):
             if getattr(position, "amplitude", 1.0) != 1.0:
                 raise ValueError("a rotation with an amplitude is not built for this mixer")
             self.inv_freq, self.pairing = rot[0], _PAIRING_CODE[rot[1]]
+            self.inv_freq_low = getattr(position, "inv_freq_low", None)
             self.rot_dims = 2 * rot[0].numel()
             if self.rot_dims > key_dim:
                 raise ValueError(f"{self.rot_dims} rotated elements exceed the key size {key_dim}")
@@ -83,6 +84,6 @@ class ConvAttention(ColumnMixer, PagedAttention):
                      positions=ctx.positions, row_req=ctx.row_request, row_offsets=ctx.row_offsets,
                      state_slots=ctx.state_slots, block_table=table, nq=nq, nkv=self.num_kv_heads, D=self.head_dim,
                      key_dim=self.key_dim, value_dim=self.value_dim, page_size=slot.page_size, inv_freq=self.inv_freq,
-                     rot_dims=self.rot_dims, pairing=self.pairing)
+                     inv_freq_low=self.inv_freq_low, rot_dims=self.rot_dims, pairing=self.pairing)
         o = self._attend(ctx, slot, plan, table, q)
         ops.gate_heads(o, proj[:, C: C + nq], out, heads=nq, D=self.head_dim, dv=self.value_dim, scale=scale)

@@ -420,6 +420,7 @@ class MoESoftmaxGroups(FeedForward):
     wants_fp32_input = True
     graph_safe = True
     adds_to = True
+    joins = True              # ``add_to`` may come from another stream (``add_ready``)
 
     def __init__(self, *, router: torch.Tensor, experts_gate_up: GroupedLinear, experts_down: GroupedLinear, top_k: int,
                  identity: int = 0, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
@@ -449,7 +450,7 @@ class MoESoftmaxGroups(FeedForward):
                              and experts_gate_up.in_features % 8 == 0 and experts_down.in_features % 8 == 0)
 
     def forward(self, ctx: StepContext, h: torch.Tensor, h32: Optional[torch.Tensor] = None,
-                add_to: Optional[torch.Tensor] = None) -> torch.Tensor:
+                add_to: Optional[torch.Tensor] = None, add_ready=None) -> torch.Tensor:
         T, k, E = h.shape[0], self.top_k, self.num_experts
         if h32 is None:
             h32 = h.to(torch.float32)
@@ -489,4 +490,6 @@ class MoESoftmaxGroups(FeedForward):
                         scale_rows=sorted_pairs)
         if side is not None:
             main.wait_stream(side)
+        if add_ready is not None:
+            main.wait_stream(add_ready)
         return ops.moe_combine_full(y, expert, weight, h32, E, shared=shared, gate=gate, add=add_to, out=add_to)

@@ -79,6 +79,15 @@ def leading_rotary_inv_freq(rot_dims: int, base: float) -> torch.Tensor:
     return torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / float(max(rot_dims, 1))).to(torch.float32)
 
 
+def leading_rotary_inv_freq_parts(rot_dims: int, base: float) -> Tuple[torch.Tensor, torch.Tensor]:
+    """:func:`leading_rotary_inv_freq` and what its rounding to float32 left out, also float32: their sum is the frequency to
+    48 bits, for kernels that form the angle of a far position with a compensated product."""
+    high = leading_rotary_inv_freq(rot_dims, base)
+    i = torch.arange(rot_dims // 2, dtype=torch.float64)
+    exact = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / float(max(rot_dims, 1)))
+    return high, (exact - high.to(torch.float64)).to(torch.float32)
+
+
 def yarn_inv_freq(rot_dims: int, base: float, factor: float, original: float, fast: float, slow: float):
     """Frequencies and amplitude of a rotation whose long waves are stretched ("YaRN"): float32 ``[rot_dims / 2]`` and
     a float.  With ``f_i = base^(-2i / rot_dims)`` and ``at(t) = rot_dims * ln(original / (2 pi t)) / (2 ln base)`` (the
@@ -110,11 +119,12 @@ def yarn_inv_freq(rot_dims: int, base: float, factor: float, original: float, fa
 @register_part("position", "rotary")
 class RotaryEncoding(PositionEncoding):
     def __init__(self, inv_freq: torch.Tensor, pairing: str = "interleaved", rot_dims: Optional[int] = None,
-                 amplitude: float = 1.0):
+                 amplitude: float = 1.0, inv_freq_low: Optional[torch.Tensor] = None):
         """``rot_dims``: only the first ``rot_dims`` elements of a head are turned, paired among themselves
         (``halves``: ``(i, i + rot_dims / 2)``; ``interleaved``: ``(2i, 2i + 1)``), and ``inv_freq`` has
         ``rot_dims / 2`` entries; None: the whole head, ``inv_freq`` of half the head size.  ``amplitude``
-        multiplies every cosine and sine (:func:`yarn_inv_freq`); the mixers that take it say so."""
+        multiplies every cosine and sine (:func:`yarn_inv_freq`); the mixers that take it say so.  ``inv_freq_low``:
+        the frequencies' low parts (:func:`leading_rotary_inv_freq_parts`), used where a kernel takes them."""
         if pairing not in ("interleaved", "halves"):
             raise ValueError(f"rotary pairing '{pairing}' is not one of interleaved, halves")
         if rot_dims is not None and (rot_dims % 2 or inv_freq.numel() != rot_dims // 2):
@@ -123,6 +133,7 @@ class RotaryEncoding(PositionEncoding):
         self.pairing = pairing
         self.rot_dims = rot_dims
         self.amplitude = float(amplitude)
+        self.inv_freq_low = inv_freq_low
 
     def rotary(self) -> Optional[Tuple[torch.Tensor, str]]:
         return self.inv_freq, self.pairing

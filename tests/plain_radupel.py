@@ -148,14 +148,18 @@ def allowed_experts(choice, count, keep):
     return ok.repeat_interleave(N // count, dim=1)
 
 
-def router_scores(h, router, t, p):
-    """(softmax scores [n, N], choice scores with minus infinity outside the kept groups)."""
+def router_scores(h, t, p):
+    """(softmax scores [n, N], choice scores [n, N])."""
     s = torch.softmax(h @ t[p + "router"].T, dim=-1)
-    choice = s + t[p + "correction"]
+    return s, s + t[p + "correction"]
+
+
+def choose(choice, router):
+    """The ``top`` experts with the largest choice scores among those of the kept groups: [n, top]."""
     groups = router.get("groups")
     if groups:
         choice = choice.masked_fill(~allowed_experts(choice, groups["count"], groups["keep"]), -math.inf)
-    return s, choice
+    return torch.topk(choice, router["top"], dim=-1).indices
 
 
 def mixture(h, mlp, t, p, round_to=None, choices=None):
@@ -163,9 +167,9 @@ def mixture(h, mlp, t, p, round_to=None, choices=None):
     Returns (output, chosen [n, top], choice scores [n, N])."""
     router = mlp["router"]
     E, ident, limit = router["experts"], router.get("identity", 0), mlp["expert"]["limit"]
-    s, choice = router_scores(h, router, t, p)
+    s, choice = router_scores(h, t, p)
     assert s.shape[1] == E + ident
-    idx = torch.topk(choice, router["top"], dim=-1).indices if choices is None else choices.to(torch.long)
+    idx = choose(choice, router) if choices is None else choices.to(torch.long)
     w = torch.gather(s, 1, idx)
     w = w / (w.sum(dim=-1, keepdim=True) + 1e-20) * router.get("scale", 1.0)
     hr = _r(h, round_to)
