@@ -517,7 +517,7 @@ def lightning(ns) -> None:
         it["i"] += 1
         y = ops.lightning(proj, col_q=cq, col_k=ck, col_v=cv, powers=powers, row_offsets=offs, state_slots=slots, state=state,
                           heads=heads, d=d, dv=dv, num_requests=B, walk_requests=dev["walk"], num_walk=plan.values["num_walk"],
-                          chunks=dev["chunks"], spans=dev["spans"])
+                          chunks=dev["chunks"], spans=dev["spans"], fast_activations=True)
         ops.norm_sigmoid_gate(y, proj[:, cg: cg + heads * dv], w, 1e-6, out)
     ms = _time(fn, max(ns.iters, copies))
     print(f"lightning batch={B} tokens={n} heads={heads} d={d} dv={dv}{' walked' if ns.walk else ''}: {ms * 1e3:.1f} us, state "

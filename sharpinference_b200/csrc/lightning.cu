@@ -29,7 +29,11 @@ constexpr int LIN_CHUNK = 64;            // rows of a chunk
 constexpr int LIN_LD = 68;               // floats between two rows of a tile in shared memory
 constexpr int LIN_MAX_KEY = 512;
 
-__device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
+// silu with the exact exponential and division, or (FAST, where the activations only have to hold up to bfloat16) with the
+// hardware's: a relative error of about 2^-21
+template <bool FAST> __device__ __forceinline__ float silu_f32(float z) {
+    return FAST ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));
+}
 
 struct LinArgs {
     const float* proj;          // [T, ld]: q at col_q (heads * d), k at col_k (heads * d), v at col_v (heads * dv)
@@ -41,6 +45,7 @@ struct LinArgs {
     long long state_stride;
     float* y;                   // [T, heads * dv]
     int heads, d, dv;
+    int fast;                   // activations with the hardware's exponential
     const int* requests;        // walk: the requests to serve (null: all)
     const int* chunks;          // chunks: [n, 4] first row, rows, request, -
     const int* spans;           // chunks: [m, 4] request, first chunk, number of chunks, -
@@ -71,7 +76,7 @@ template <int VEC> __device__ __forceinline__ void store_pack(float* p, const Pa
     else *p = r.v[0];
 }
 
-template <int ROWS, int VEC>             // state rows a warp (8 ROWS >= d), columns a lane
+template <bool FAST, int ROWS, int VEC>  // state rows a warp (8 ROWS >= d), columns a lane
 __global__ void __launch_bounds__(LIN_THREADS) lightning_walk_kernel(LinArgs a) {
     constexpr int COLS = 32 * VEC;
     __shared__ __align__(16) float q_s[LIN_STAGE][LIN_WARPS * ROWS];
@@ -108,12 +113,12 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_walk_kernel(LinArgs a) 
         for (int i = threadIdx.x; i < nr * LIN_WARPS * ROWS; i += LIN_THREADS) {
             const int r = i / (LIN_WARPS * ROWS), n = i % (LIN_WARPS * ROWS);
             const float* row = src + (size_t)r * a.ld + (size_t)h * d + n;
-            q_s[r][n] = n < d ? silu_f32(row[a.col_q]) : 0.0f;
-            k_s[r][n] = n < d ? silu_f32(row[a.col_k]) : 0.0f;
+            q_s[r][n] = n < d ? silu_f32<FAST>(row[a.col_q]) : 0.0f;
+            k_s[r][n] = n < d ? silu_f32<FAST>(row[a.col_k]) : 0.0f;
         }
         for (int i = threadIdx.x; i < nr * COLS; i += LIN_THREADS) {
             const int r = i / COLS, cc = c0 + i % COLS;
-            v_s[r][i % COLS] = cc < dv ? silu_f32(src[(size_t)r * a.ld + a.col_v + (size_t)h * dv + cc]) : 0.0f;
+            v_s[r][i % COLS] = cc < dv ? silu_f32<FAST>(src[(size_t)r * a.ld + a.col_v + (size_t)h * dv + cc]) : 0.0f;
         }
         __syncthreads();
         for (int r = 0; r < nr; ++r) {
@@ -151,9 +156,9 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_walk_kernel(LinArgs a) 
 
 template <int ROWS, int VEC>
 static int launch_walk(const LinArgs& a, int n, cudaStream_t stream) {
-    auto kern = lightning_walk_kernel<ROWS, VEC>;
     const dim3 grid((a.dv + 32 * VEC - 1) / (32 * VEC), a.heads, n);
-    SHARPI_LAUNCH_PDL(kern, grid, LIN_THREADS, 0, stream, a);
+    if (a.fast) SHARPI_LAUNCH_PDL((lightning_walk_kernel<true, ROWS, VEC>), grid, LIN_THREADS, 0, stream, a);
+    else SHARPI_LAUNCH_PDL((lightning_walk_kernel<false, ROWS, VEC>), grid, LIN_THREADS, 0, stream, a);
     return SHARPI_OK;
 }
 
@@ -173,13 +178,13 @@ static bool fill_args(LinArgs& a, const float* proj, int ld, int col_q, int col_
 SHARPI_API int sharpi_lightning_walk(const float* proj, int ld, int col_q, int col_k, int col_v, const float* pow,
                                      const int* row_offsets, const int* state_slots, const int* requests, int n,
                                      float* state, long long state_stride, float* y, int heads, int d, int dv,
-                                     cudaStream_t stream) {
+                                     int fast, cudaStream_t stream) {
     if (n <= 0) return SHARPI_OK;
     LinArgs a;
     if (n > 65535 || !fill_args(a, proj, ld, col_q, col_k, col_v, pow, row_offsets, state_slots, state, state_stride, y,
                                 heads, d, dv))
         return SHARPI_BAD_ARGUMENT;
-    a.requests = requests;
+    a.requests = requests; a.fast = fast;
     const bool al4 = dv % 4 == 0 && state_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
     const bool al2 = dv % 2 == 0 && state_stride % 2 == 0 && (reinterpret_cast<uintptr_t>(state) & 7) == 0;
     const int vec = (al4 && dv > 64) ? 4 : (al2 && dv > 32) ? 2 : 1;
@@ -193,28 +198,36 @@ SHARPI_API int sharpi_lightning_walk(const float* proj, int ld, int col_q, int c
 // -------------------------------------------------------------------------------------------------------------
 // chunks
 // -------------------------------------------------------------------------------------------------------------
-// A 64 x 64 tile of columns c .. c + 63 (those below `cols`; zeros behind) of rows row0 .. row0 + rows - 1 (zeros behind),
-// through silu where ACT.
-template <bool ACT>
-__device__ __forceinline__ void load_tile(float* dst, const float* src, size_t ld, int c, int cols, int rows, bool vec) {
+// A 64 x 64 tile of columns c .. c + 63 (those below `cols`; zeros behind) of rows row0 .. row0 + rows - 1 (zeros behind):
+// as it is (ACT 0), through silu (1: exact, 2: fast), and times pw[rows - 1 - row] where `pw` is given.
+template <int ACT>
+__device__ __forceinline__ float tile_value(float x, float f) {
+    return ACT == 0 ? x : f * silu_f32<ACT == 2>(x);
+}
+
+template <int ACT>
+__device__ __forceinline__ void load_tile(float* dst, const float* src, size_t ld, int c, int cols, int rows, bool vec,
+                                          const float* pw = nullptr) {
     if (vec) {
-        for (int i = threadIdx.x; i < LIN_CHUNK * 16; i += LIN_THREADS) {
-            const int r = i >> 4, e = (i & 15) * 4;
-            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (r < rows && c + e < cols) {
-                x = *reinterpret_cast<const float4*>(src + (size_t)r * ld + c + e);
-                if (ACT) x = make_float4(silu_f32(x.x), silu_f32(x.y), silu_f32(x.z), silu_f32(x.w));
-            }
-            *reinterpret_cast<float4*>(dst + r * LIN_LD + e) = x;
+        float4 x[4];                                           // all four pieces of a thread are asked for at once
+#pragma unroll
+        for (int p = 0; p < 4; ++p) {
+            const int i = threadIdx.x + p * LIN_THREADS, r = i >> 4, e = (i & 15) * 4;
+            x[p] = r < rows && c + e < cols ? *reinterpret_cast<const float4*>(src + (size_t)r * ld + c + e)
+                                            : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+#pragma unroll
+        for (int p = 0; p < 4; ++p) {
+            const int i = threadIdx.x + p * LIN_THREADS, r = i >> 4, e = (i & 15) * 4;
+            const float f = pw && r < rows ? pw[rows - 1 - r] : 1.0f;
+            *reinterpret_cast<float4*>(dst + r * LIN_LD + e) = make_float4(
+                tile_value<ACT>(x[p].x, f), tile_value<ACT>(x[p].y, f), tile_value<ACT>(x[p].z, f), tile_value<ACT>(x[p].w, f));
         }
     } else {
         for (int i = threadIdx.x; i < LIN_CHUNK * 64; i += LIN_THREADS) {
             const int r = i >> 6, e = i & 63;
             float x = 0.0f;
-            if (r < rows && c + e < cols) {
-                x = src[(size_t)r * ld + c + e];
-                if (ACT) x = silu_f32(x);
-            }
+            if (r < rows && c + e < cols) x = tile_value<ACT>(src[(size_t)r * ld + c + e], pw ? pw[rows - 1 - r] : 1.0f);
             dst[r * LIN_LD + e] = x;
         }
     }
@@ -265,6 +278,7 @@ __device__ __forceinline__ void tile_mul_t(const float* A, const float* B, int t
 }
 
 // (1) sums[chunk][h][n][v] = sum_i a^(rows - 1 - i) k_i[n] v_i[v]; a block makes 64 x 64 of them
+template <bool FAST>
 __global__ void __launch_bounds__(LIN_THREADS) lightning_sums_kernel(LinArgs a, int tiles_v, int vec) {
     __shared__ __align__(16) float k_s[LIN_CHUNK * LIN_LD];
     __shared__ __align__(16) float v_s[LIN_CHUNK * LIN_LD];
@@ -273,11 +287,8 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_sums_kernel(LinArgs a, 
     const int n0 = (blockIdx.x / tiles_v) * 64, c0 = (blockIdx.x % tiles_v) * 64;
     const int row0 = a.chunks[4 * chunk], rows = a.chunks[4 * chunk + 1];
     const float* src = a.proj + (size_t)row0 * a.ld;
-    load_tile<true>(k_s, src + a.col_k + (size_t)h * a.d, a.ld, n0, a.d, rows, vec);
-    load_tile<true>(v_s, src + a.col_v + (size_t)h * a.dv, a.ld, c0, a.dv, rows, vec);
-    __syncthreads();
-    const float* pw = a.pow + h * (LIN_CHUNK + 1);
-    for (int i = threadIdx.x; i < rows * 64; i += LIN_THREADS) k_s[(i >> 6) * LIN_LD + (i & 63)] *= pw[rows - 1 - (i >> 6)];
+    load_tile<FAST ? 2 : 1>(k_s, src + a.col_k + (size_t)h * a.d, a.ld, n0, a.d, rows, vec, a.pow + h * (LIN_CHUNK + 1));
+    load_tile<FAST ? 2 : 1>(v_s, src + a.col_v + (size_t)h * a.dv, a.ld, c0, a.dv, rows, vec);
     __syncthreads();
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
     float acc[4][4] = {};
@@ -324,7 +335,7 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_carry_kernel(LinArgs a)
     const size_t step = (size_t)a.heads * size;
     float* u = a.sums + (size_t)chunk0 * step + (size_t)h * size + i;
     Pack<VEC> S = load_pack<VEC>(st);
-    constexpr int AHEAD = 4;                                   // chunk sums asked for ahead of the walk
+    constexpr int AHEAD = 8;                                   // chunk sums asked for ahead of the walk
     Pack<VEC> next[AHEAD];
 #pragma unroll
     for (int k = 0; k < AHEAD; ++k)
@@ -345,7 +356,8 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_carry_kernel(LinArgs a)
 }
 
 // (3) the outputs of one chunk's rows, 64 value columns of one head
-__global__ void __launch_bounds__(LIN_THREADS) lightning_out_kernel(LinArgs a, int vec) {
+template <bool FAST>
+__global__ void __launch_bounds__(LIN_THREADS, 3) lightning_out_kernel(LinArgs a, int vec) {
     extern __shared__ __align__(16) float lin_smem[];
     float* q_s = lin_smem;
     float* k_s = q_s + LIN_CHUNK * LIN_LD;
@@ -358,18 +370,19 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_out_kernel(LinArgs a, i
     const float* before = a.sums + ((size_t)chunk * a.heads + h) * a.d * a.dv;
     if (threadIdx.x <= LIN_CHUNK) pw[threadIdx.x] = a.pow[h * (LIN_CHUNK + 1) + threadIdx.x];
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    constexpr int ACT = FAST ? 2 : 1;
     float score[4][4] = {}, past[4][4] = {};
     for (int n0 = 0; n0 < a.d; n0 += 64) {
         if (n0) __syncthreads();
-        load_tile<true>(q_s, src + a.col_q + (size_t)h * a.d, a.ld, n0, a.d, rows, vec);
-        load_tile<true>(k_s, src + a.col_k + (size_t)h * a.d, a.ld, n0, a.d, rows, vec);
-        load_tile<false>(s_s, before + (size_t)n0 * a.dv, a.dv, c0, a.dv, min(64, a.d - n0), vec);
+        load_tile<ACT>(q_s, src + a.col_q + (size_t)h * a.d, a.ld, n0, a.d, rows, vec);
+        load_tile<ACT>(k_s, src + a.col_k + (size_t)h * a.d, a.ld, n0, a.d, rows, vec);
+        load_tile<0>(s_s, before + (size_t)n0 * a.dv, a.dv, c0, a.dv, min(64, a.d - n0), vec);
         __syncthreads();
         tile_mul_t(q_s, k_s, ty, tx, score);
         tile_mul(q_s, s_s, ty, tx, past);
     }
     __syncthreads();
-    load_tile<true>(k_s, src + a.col_v + (size_t)h * a.dv, a.ld, c0, a.dv, rows, vec);        // the values
+    load_tile<ACT>(k_s, src + a.col_v + (size_t)h * a.dv, a.ld, c0, a.dv, rows, vec);         // the values
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -403,22 +416,24 @@ __global__ void __launch_bounds__(LIN_THREADS) lightning_out_kernel(LinArgs a, i
 SHARPI_API int sharpi_lightning_chunks(const float* proj, int ld, int col_q, int col_k, int col_v, const float* pow,
                                        const int* row_offsets, const int* state_slots, const int* chunks, int n_chunks,
                                        const int* spans, int n_spans, float* sums, float* state, long long state_stride,
-                                       float* y, int heads, int d, int dv, cudaStream_t stream) {
+                                       float* y, int heads, int d, int dv, int fast, cudaStream_t stream) {
     if (n_chunks <= 0) return SHARPI_OK;
     LinArgs a;
     if (n_chunks > 65535 || n_spans <= 0 || n_spans > 65535 ||
         !fill_args(a, proj, ld, col_q, col_k, col_v, pow, row_offsets, state_slots, state, state_stride, y, heads, d, dv))
         return SHARPI_BAD_ARGUMENT;
-    a.chunks = chunks; a.spans = spans; a.sums = sums;
+    a.chunks = chunks; a.spans = spans; a.sums = sums; a.fast = fast;
     const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(sums) |
                            reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(y);
     const int vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && col_q % 4 == 0 && col_k % 4 == 0 && col_v % 4 == 0 &&
                     state_stride % 4 == 0 && (ptrs & 15) == 0;
     const int tiles_n = (d + 63) / 64, tiles_v = (dv + 63) / 64;
-    SHARPI_LAUNCH_PDL(lightning_sums_kernel, dim3(tiles_n * tiles_v, heads, n_chunks), LIN_THREADS, 0, stream, a, tiles_v, vec);
+    const dim3 sum_grid(tiles_n * tiles_v, heads, n_chunks);
+    if (fast) SHARPI_LAUNCH_PDL(lightning_sums_kernel<true>, sum_grid, LIN_THREADS, 0, stream, a, tiles_v, vec);
+    else SHARPI_LAUNCH_PDL(lightning_sums_kernel<false>, sum_grid, LIN_THREADS, 0, stream, a, tiles_v, vec);
     const int size = d * dv;
     if (vec)
-        SHARPI_LAUNCH_PDL(lightning_carry_kernel<4>, dim3((size / 4 + LIN_THREADS - 1) / LIN_THREADS, heads, n_spans),
+        SHARPI_LAUNCH_PDL(lightning_carry_kernel<2>, dim3((size / 2 + LIN_THREADS - 1) / LIN_THREADS, heads, n_spans),
                           LIN_THREADS, 0, stream, a);
     else
         SHARPI_LAUNCH_PDL(lightning_carry_kernel<1>, dim3((size + LIN_THREADS - 1) / LIN_THREADS, heads, n_spans),
@@ -426,11 +441,13 @@ SHARPI_API int sharpi_lightning_chunks(const float* proj, int ld, int col_q, int
     constexpr size_t smem = (3 * LIN_CHUNK * LIN_LD + LIN_CHUNK + 4) * sizeof(float);
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(lightning_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(lightning_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(lightning_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return SHARPI_LAUNCH_FAILED;
         configured = true;
     }
-    SHARPI_LAUNCH_PDL(lightning_out_kernel, dim3(tiles_v, heads, n_chunks), LIN_THREADS, smem, stream, a, vec);
+    if (fast) SHARPI_LAUNCH_PDL(lightning_out_kernel<true>, dim3(tiles_v, heads, n_chunks), LIN_THREADS, smem, stream, a, vec);
+    else SHARPI_LAUNCH_PDL(lightning_out_kernel<false>, dim3(tiles_v, heads, n_chunks), LIN_THREADS, smem, stream, a, vec);
     return SHARPI_OK;
 }
 

@@ -89,8 +89,8 @@ SIGNATURES: Dict[str, Tuple[str, list]] = {
     "sharpi_gate_heads": ("elementwise", [P, P, I, P, I, I, I, I, I, I, F, P]),
     "sharpi_softcap": ("elementwise", [P, F, LL, P]),
     "sharpi_qkv_conv": ("rope_kv", [P, I, I, P, I, P, LL, P, P, P, P, P, P, P, I, I, P, P, I, I, I, I, I, I, I, I, I, P]),
-    "sharpi_lightning_walk": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, LL, P, I, I, I, P]),
-    "sharpi_lightning_chunks": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, I, P, P, LL, P, I, I, I, P]),
+    "sharpi_lightning_walk": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, LL, P, I, I, I, I, P]),
+    "sharpi_lightning_chunks": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, I, P, P, LL, P, I, I, I, I, P]),
     "sharpi_norm_sigmoid_gate": ("lightning", [P, P, I, P, F, F, I, I, P, I, I, P]),
     "sharpi_router_groups": ("moe_topk", [P, P, P, I, I, I, I, F, I, I, I, P, P, P, P, P, P]),
     "sharpi_moe_combine_full": ("moe_topk", [P, P, P, P, P, P, P, P, I, I, I, I, P]),

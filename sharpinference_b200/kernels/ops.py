@@ -1628,11 +1628,13 @@ def decay_powers(decay) -> torch.Tensor:
 def lightning(proj: torch.Tensor, *, col_q: int, col_k: int, col_v: int, powers: torch.Tensor, row_offsets: torch.Tensor,
               state_slots: torch.Tensor, state: torch.Tensor, heads: int, d: int, dv: int, num_requests: int,
               walk_requests: Optional[torch.Tensor] = None, num_walk: Optional[int] = None,
-              chunks: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None) -> torch.Tensor:
+              chunks: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None,
+              fast_activations: bool = False) -> torch.Tensor:
     """``S <- a S + silu(k) silu(v)^T``, ``o = S^T silu(q)`` per head for the step's rows; float32 ``[T, heads * dv]``.
     ``proj`` float32 ``[T, *]`` (a column range) holds q, k and v at the named columns; ``state`` float32
     ``[slots, heads * d * dv]``.  ``walk_requests`` (None: all ``num_requests``) are walked row by row; the requests of
-    ``spans`` (int32 ``[m, 4]``) by chunks (int32 ``[n, 4]``, at most LIGHTNING_CHUNK rows each)."""
+    ``spans`` (int32 ``[m, 4]``) by chunks (int32 ``[n, 4]``, at most LIGHTNING_CHUNK rows each).  ``fast_activations``: silu
+    with the hardware's exponential and division (relative error about 2^-21), where they need not be float32 exact."""
     ld = _need_columns(proj, "proj", torch.float32)
     _need(powers, "powers", torch.float32)
     _need(state, "state", torch.float32)
@@ -1653,15 +1655,15 @@ def lightning(proj: torch.Tensor, *, col_q: int, col_k: int, col_v: int, powers:
         check(kernel("sharpi_lightning_chunks")(proj.data_ptr(), ld, col_q, col_k, col_v, powers.data_ptr(),
                                                 row_offsets.data_ptr(), state_slots.data_ptr(), chunks.data_ptr(),
                                                 chunks.shape[0], spans.data_ptr(), spans.shape[0], sums.data_ptr(),
-                                                state.data_ptr(), state.stride(0), y.data_ptr(), heads, d, dv, _stream()),
-              "sharpi_lightning_chunks")
+                                                state.data_ptr(), state.stride(0), y.data_ptr(), heads, d, dv, int(fast_activations),
+                                                _stream()), "sharpi_lightning_chunks")
     if n_walk:
         if walk_requests is not None:
             _need(walk_requests, "walk_requests", torch.int32)
         check(kernel("sharpi_lightning_walk")(proj.data_ptr(), ld, col_q, col_k, col_v, powers.data_ptr(),
                                               row_offsets.data_ptr(), state_slots.data_ptr(), _ptr(walk_requests), n_walk,
-                                              state.data_ptr(), state.stride(0), y.data_ptr(), heads, d, dv, _stream()),
-              "sharpi_lightning_walk")
+                                              state.data_ptr(), state.stride(0), y.data_ptr(), heads, d, dv, int(fast_activations),
+                                              _stream()), "sharpi_lightning_walk")
     return y
 
 

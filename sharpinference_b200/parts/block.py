@@ -26,7 +26,7 @@ from .base import Block, ColumnMixer, FeedForward, LayerSlot, Mixer, Norm, StepC
 from .branches import side_by_side, pad_columns
 from .linear import Linear
 from .norm import RMSNorm
-from .side import fork
+from .side import fork, join
 
 
 @register_part("block", "prenorm")
@@ -89,7 +89,7 @@ class ParallelPairBlock(Block):
             return x, self.mixer.forward(ctx, slot, h)
         h1, h2, h32 = self._norms(x, pending, self.ffn.wants_fp32_input)
         # the mixer and the feed-forward meet in the last product or sum: the mixer runs on a stream of its own
-        main, side = torch.cuda.current_stream(x.device), fork(x.device, "mixer")
+        side = fork(x.device, "mixer", ctx.decode_only)
         if self.joint_out is not None:
             cols = torch.empty((x.shape[0], self.joint_out.in_features), dtype=self.act_dtype, device=x.device)
             with torch.cuda.stream(side):
@@ -97,12 +97,12 @@ class ParallelPairBlock(Block):
                     cols[:, self.mixer.out_columns: self._ffn_at].zero_()
                 self.mixer.inner_from(ctx, slot, h1, cols[:, : self.mixer.out_columns])
             self.ffn.inner(ctx, h2, cols[:, self._ffn_at:])
-            main.wait_stream(side)
+            join(side)
             return x, self.joint_out(cols)
         with torch.cuda.stream(side):
             mixed = self.mixer.forward(ctx, slot, h1)
         if getattr(self.ffn, "joins", False):              # adds the mixer's output in its last kernel, and waits for it there
             return x, self.ffn.forward(ctx, h2, h32, add_to=mixed, add_ready=side)
         y = self.ffn.forward(ctx, h2, h32)
-        main.wait_stream(side)
+        join(side)
         return x, ops.add(mixed, y, out=mixed)

@@ -16,7 +16,7 @@ import torch
 from .base import ColumnMixer, LayerSlot, StepContext, StepPlanner, register_part
 from .linear import Linear
 from .mamba import BranchPair
-from .side import fork
+from .side import fork, join
 
 
 def pad_columns(n: int) -> int:
@@ -69,9 +69,9 @@ class ScaledBranches(ColumnMixer):
 
     def inner(self, ctx: StepContext, slot: LayerSlot, proj: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
         # the branches meet in the output product: the right one runs on a stream of its own
-        side = fork(proj.device, "branch")
+        side = fork(proj.device, "branch", ctx.decode_only)
         with torch.cuda.stream(side):
             self._branch(ctx, slot, self.right, "right.", proj, out, self.left.in_columns, self._right_at,
                          scale * self.right_scale)
         self._branch(ctx, slot, self.left, "left.", proj, out, 0, 0, scale * self.left_scale)
-        torch.cuda.current_stream(proj.device).wait_stream(side)
+        join(side)

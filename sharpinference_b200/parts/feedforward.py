@@ -22,6 +22,7 @@ import torch
 from ..kernels import ops
 from .base import FeedForward, StepContext, register_part
 from .linear import GroupedLinear, Linear
+from .side import fork, join
 
 
 @register_part("feed_forward", "dense_swiglu")
@@ -455,11 +456,9 @@ class MoESoftmaxGroups(FeedForward):
         if h32 is None:
             h32 = h.to(torch.float32)
         # the shared expert meets the routed ones only in the last sum: it runs on a second stream meanwhile
-        main = torch.cuda.current_stream(h.device)
         shared = side = None
         if self.shared is not None:
-            side = _side_stream(h.device)
-            side.wait_stream(main)
+            side = fork(h.device, "shared", ctx.decode_only)
             with torch.cuda.stream(side):
                 shared = self.shared.forward(ctx, h)
         expert, weight, gate, _ = ops.router_groups(h32, self.router, k, correction=self.correction, scale=self.route_scale,
@@ -489,7 +488,7 @@ class MoESoftmaxGroups(FeedForward):
             ops.gemm_nt(act, w_down, out=y, group_offsets=offsets, out_rows=sorted_pairs, rows=T * k, row_scale=w_pairs,
                         scale_rows=sorted_pairs)
         if side is not None:
-            main.wait_stream(side)
+            join(side)
         if add_ready is not None:
-            main.wait_stream(add_ready)
+            join(add_ready)
         return ops.moe_combine_full(y, expert, weight, h32, E, shared=shared, gate=gate, add=add_to, out=add_to)

@@ -34,7 +34,7 @@ class LightningPlanner(StepPlanner):
     ``chunks`` ``[n, 4]`` (first row, rows, request, 0), a request's one after the other, and ``spans`` ``[m, 4]``
     (request, first chunk, chunks, 0).  Which of the two a request is depends on its own rows alone."""
 
-    WALK_ROWS_UP_TO = 16
+    WALK_ROWS_UP_TO = 32        # (one head of 128 x 128 a block: 31 us walked, 44 us as a chunk)
     key = ("lightning",)
 
     def plan(self, starts: Sequence[int], lengths: Sequence[int], bucket: Hashable = None) -> StepPlanData:
@@ -92,6 +92,7 @@ class LightningAttention(ColumnMixer):
         y = ops.lightning(proj, col_q=self.col_q, col_k=self.col_k, col_v=self.col_v, powers=self.powers,
                           row_offsets=ctx.row_offsets, state_slots=ctx.state_slots, state=slot.states["S"],
                           heads=self.heads, d=self.dim, dv=self.value_dim, num_requests=ctx.num_requests,
-                          walk_requests=plan.walk, num_walk=plan.num_walk, chunks=plan.chunks, spans=plan.spans)
+                          walk_requests=plan.walk, num_walk=plan.num_walk, chunks=plan.chunks, spans=plan.spans,
+                          fast_activations=self.act_dtype == torch.bfloat16)
         n = self.heads * self.value_dim
         ops.norm_sigmoid_gate(y, proj[:, self.col_g: self.col_g + n], self.norm_weight, self.eps, out, scale=scale)

@@ -288,17 +288,18 @@ def test_angles_of_far_positions():
     assert err["with"] < 2e-6 and err["without"] > 1e-3, err
 
 
+@pytest.mark.parametrize("fast", [False, True])
 @pytest.mark.parametrize("H,d,dv,decay", [(2, 32, 32, (0.6, 0.999)), (3, 5, 7, (0.7, 0.0, 1.0)), (1, 128, 128, (0.995,)),
                                           (2, 64, 40, (0.9, 0.99)), (1, 160, 72, (0.98,)), (1, 300, 24, (0.97,)), (2, 1, 1, (0.5, 0.9)),
                                           (1, 96, 200, (0.9,)), (2, 128, 64, (0.3, 0.9999))])
-def test_decayed_sums_walked_and_in_chunks(H, d, dv, decay):
+def test_decayed_sums_walked_and_in_chunks(H, d, dv, decay, fast):
     """Three requests on slots of their own, in portions of one to 150 rows, walked and in chunks of 64 (also a last chunk of
     one row), against the sums row by row; the two forms continue one another's state."""
     from sharpinference_b200.kernels import ops
     from sharpinference_b200.parts import LightningPlanner
     cols = 2 * H * d + H * dv
     powers = ops.decay_powers(decay).to(DEV)
-    sizes = [[150, 3, 65, 1], [1, 129, 2, 17], [40, 16, 1, 64]]
+    sizes = [[150, 3, 65, 1], [1, 129, 2, 33], [40, 32, 1, 64]]
     n = [sum(s) for s in sizes]
     us = [_rand(m, cols, seed=70 + i) for i, m in enumerate(n)]
     slots = [3, 0, 2]
@@ -315,7 +316,8 @@ def test_decayed_sums_walked_and_in_chunks(H, d, dv, decay):
         dev = {k: (torch.from_numpy(v).to(DEV) if v.size else None) for k, v in plan.arrays.items()}
         y = ops.lightning(f32(proj), col_q=4, col_k=4 + H * d, col_v=4 + 2 * H * d, powers=powers, row_offsets=i32(off),
                           state_slots=i32(slots), state=state, heads=H, d=d, dv=dv, num_requests=3, walk_requests=dev["walk"],
-                          num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"]).cpu()
+                          num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"],
+                          fast_activations=fast).cpu()
         for b in range(3):
             got[b].append(y[off[b]: off[b + 1]])
             at[b] += lens[b]
@@ -500,7 +502,7 @@ def test_portions_down_to_two_tokens(folders, expected, name, dtype):
     """Portions shorter and longer than the convolutions' memory, at and around the size from which the linear attention works
     in chunks, and across chunk borders."""
     run_and_compare(folders[name], name, dtype, traces.portions(requests_for(name)), expected)
-    run_and_compare(folders[name], name, dtype, traces.portions(requests_for(name), sizes=(2, 17, 3, 64, 1, 16, 2, 65, 33, 2)),
+    run_and_compare(folders[name], name, dtype, traces.portions(requests_for(name), sizes=(2, 17, 3, 64, 1, 32, 2, 65, 33, 2)),
                     expected, page_size=16)
 
 
