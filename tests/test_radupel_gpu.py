@@ -735,9 +735,37 @@ def test_command_line_and_trace_program(folders, capsys, tmp_path):
             at[e["id"]] += len(e["tokens"])
 
 
-def test_parts_are_registered_and_column_mixers_run_alone(folders):
-    """A branch by itself is a mixer like any other: its own two products around its inner columns."""
+def test_parts_are_registered():
     from sharpinference_b200.parts import part_kinds
     assert {"conv_attention", "lightning_attention", "scaled_branches"} <= set(part_kinds("mixer"))
     assert "parallel_pair" in part_kinds("block") and "add_input" in part_kinds("stream")
     assert "moe_softmax_groups" in part_kinds("feed_forward")
+
+
+def test_a_branch_by_itself_is_a_mixer():
+    """Linear attention outside a pair: its own two products around its inner columns, in portions of 50, 3 and 40 rows."""
+    from types import SimpleNamespace
+
+    from sharpinference_b200.parts import LayerSlot, LightningAttention, LightningPlanner, lightning_columns
+    W, H, d, dv = 24, 3, 6, 10
+    t = {"q": _rand(H * d, W, seed=1), "k": _rand(H * d, W, seed=2), "v": _rand(H * dv, W, seed=3), "g": _rand(H * dv, W, seed=4),
+         "o": _rand(W, H * dv, seed=5), "norm": _rand(H * dv, seed=6)}
+    m = {"heads": H, "dim": d, "vdim": dv, "decay": [0.5, 0.9, 0.99]}
+    rows = torch.cat([t[s] for s in "qkvg"])
+    proj = torch.zeros(lightning_columns(H, d, dv)[-1], W, dtype=F64)
+    proj[: rows.shape[0]] = rows
+    mixer = LightningAttention(proj=f32(proj), out=f32(t["o"]), norm_weight=f32(t["norm"]), decay=m["decay"], heads=H, dim=d,
+                               value_dim=dv, eps=1e-5, act_dtype=torch.float32)
+    state = torch.zeros(2, mixer.state_specs["S"].shape[0], device=DEV)
+    slot = LayerSlot(index=0, layer=0, states={"S": state})
+    h = _rand(93, W, seed=7, scale=0.3)
+    got, at = [], 0
+    for n in (50, 3, 40):
+        data = LightningPlanner().plan([at], [n])
+        arrays = {k: (torch.from_numpy(v).to(DEV) if v.size else None) for k, v in data.arrays.items()}
+        ctx = SimpleNamespace(num_tokens=n, num_requests=1, row_offsets=i32([0, n]), state_slots=i32([1]),
+                              plans={LightningPlanner.key: SimpleNamespace(**arrays, **data.values)})
+        got.append(mixer.forward(ctx, slot, f32(h[at: at + n])).cpu())
+        at += n
+    close(torch.cat(got), plain.lightning(h, m, t, "", 1e-5), 1e-5)
+    assert float(state[0].abs().max()) == 0.0
