@@ -5,9 +5,10 @@ from .notedra import NotedraConfig, NotedraLayer, NotedraMLP
 from .gisilix import GisilixConfig, GisilixLayer, GisilixMLP, GisilixYarn
 from .latinex import LatinexConfig, LatinexLayer, LatinexMoE
 from .radupel import RadupelAttention, RadupelConfig, RadupelLayer, RadupelLinear, RadupelMLP
+from .sufopel import SufopelConfig, SufopelDelta, SufopelLatent, SufopelLayer, SufopelMLP
 from .zaposun import ZaposunAttention, ZaposunConfig, ZaposunLayer, ZaposunScan
 
 __all__ = ["ConfigError", "ConfigReader", "architecture_name", "read_config_json",
            "Llama4TextConfig", "RopeScaling", "NotedraConfig", "NotedraLayer", "NotedraMLP", "ZaposunAttention",
            "ZaposunConfig", "ZaposunLayer", "ZaposunScan", "LatinexConfig", "LatinexLayer", "LatinexMoE", "GisilixConfig", "GisilixLayer", "GisilixMLP", "GisilixYarn",
-           "RadupelAttention", "RadupelConfig", "RadupelLayer", "RadupelLinear", "RadupelMLP"]
+           "SufopelConfig", "SufopelDelta", "SufopelLatent", "SufopelLayer", "SufopelMLP", "RadupelAttention", "RadupelConfig", "RadupelLayer", "RadupelLinear", "RadupelMLP"]

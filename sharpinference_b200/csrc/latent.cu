@@ -20,7 +20,9 @@
 //
 // `ld` / `ldq`: the distance between two rows of the source when it is a column range of a wider product; `rot_amp`:
 // a factor on the rotation's cosines and sines (frequency scalings that also stretch the amplitude); `gate` of
-// head_minor: [T, gate_ld] float32 logits, head h of row t is multiplied by sigmoid(gate[t, h]).
+// head_minor: [T, gate_ld] float32 logits, head h of row t is multiplied by sigmoid(gate[t, h]), or element c of it by
+// sigmoid(gate[t, h n + c]) (`gate_elem`).  Without `write_kv` (a layer that reads another one's latents) latent_down_post
+// norms the query latent alone and the columns behind it may be absent.
 //
 // Norm sums, angles, sines and cosines are float32; a row's numbers depend on the row alone.
 #include "common.cuh"
@@ -40,9 +42,10 @@ latent_down_post_kernel(const float* down, int ld, int q_rank, int rank, int rot
     const float* row = down + (size_t)t * ld;
     float ssq = 0.0f, ssc = 0.0f;
     for (int i = threadIdx.x; i < q_rank; i += LAT_THREADS) ssq += row[i] * row[i];
-    for (int i = threadIdx.x; i < rank; i += LAT_THREADS) ssc += row[q_rank + i] * row[q_rank + i];
+    if (write_kv)
+        for (int i = threadIdx.x; i < rank; i += LAT_THREADS) ssc += row[q_rank + i] * row[q_rank + i];
     ssq = block_sum(ssq, scratch);
-    ssc = block_sum(ssc, scratch);
+    if (write_kv) ssc = block_sum(ssc, scratch);
     if (q_rank > 0) {
         const float sq = 1.0f / sqrtf(ssq / (float)q_rank + eps);
         for (int i = threadIdx.x; i < q_rank; i += LAT_THREADS)
@@ -84,8 +87,8 @@ SHARPI_API int sharpi_latent_down_post(const float* down, int ld, int q_rank, in
                                        int write_kv, int out_dtype, int T, float rot_amp, cudaStream_t stream) {
     if (T <= 0) return SHARPI_OK;
     if (q_rank < 0 || rank <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || (rot_dims & 1) ||
-        q_rank + rank + rot > ld || rank + rot > D || (kv_planes != 1 && kv_planes != 2) || page_size <= 0 ||
-        max_blocks <= 0 || (q_rank > 0 && !wq) || !wc)
+        q_rank + (write_kv ? rank + rot : 0) > ld || rank + rot > D || (kv_planes != 1 && kv_planes != 2) ||
+        page_size <= 0 || max_blocks <= 0 || (q_rank > 0 && !wq) || (write_kv && !wc))
         return SHARPI_BAD_ARGUMENT;
     if (out_dtype == SHARPI_F32)
         SHARPI_LAUNCH_PDL(latent_down_post_kernel<float>, T, LAT_THREADS, 0, stream, down, ld, q_rank, rank, rot,
@@ -134,7 +137,7 @@ SHARPI_API int sharpi_head_major(const void* src, int src_dtype, int T, int head
 template <typename TO>
 __global__ void __launch_bounds__(256)
 head_minor_kernel(const float* src, int T, int heads, int stride, int col0, int n, TO* dst, const float* gate,
-                  int gate_ld) {
+                  int gate_ld, int gate_elem) {
     pdl_wait();
     const long long total = (long long)T * heads * n;
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -143,20 +146,20 @@ head_minor_kernel(const float* src, int T, int heads, int stride, int col0, int 
     const long long th = i / n;
     const int h = (int)(th % heads), t = (int)(th / heads);
     float v = src[((size_t)h * T + t) * n + c];
-    if (gate) v = v / (1.0f + expf(-gate[(size_t)t * gate_ld + h]));      // the head's output times sigmoid(gate logit)
+    if (gate) v = v / (1.0f + expf(-gate[(size_t)t * gate_ld + (gate_elem ? h * n + c : h)]));      // times sigmoid(gate logit)
     dst[((size_t)t * heads + h) * stride + col0 + c] = from_float<TO>(v);
 }
 
 SHARPI_API int sharpi_head_minor(const float* src, int T, int heads, int stride, int col0, int n, void* dst,
-                                 int dst_dtype, const float* gate, int gate_ld, cudaStream_t stream) {
+                                 int dst_dtype, const float* gate, int gate_ld, int gate_elem, cudaStream_t stream) {
     if (T <= 0 || n <= 0) return SHARPI_OK;
     if (heads <= 0 || col0 < 0 || col0 + n > stride) return SHARPI_BAD_ARGUMENT;
     const long long total = (long long)T * heads * n;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (dst_dtype == SHARPI_F32)
-        SHARPI_LAUNCH_PDL(head_minor_kernel<float>, blocks, 256, 0, stream, src, T, heads, stride, col0, n, (float*)dst, gate, gate_ld);
+        SHARPI_LAUNCH_PDL(head_minor_kernel<float>, blocks, 256, 0, stream, src, T, heads, stride, col0, n, (float*)dst, gate, gate_ld, gate_elem);
     else if (dst_dtype == SHARPI_BF16)
-        SHARPI_LAUNCH_PDL(head_minor_kernel<bf16>, blocks, 256, 0, stream, src, T, heads, stride, col0, n, (bf16*)dst, gate, gate_ld);
+        SHARPI_LAUNCH_PDL(head_minor_kernel<bf16>, blocks, 256, 0, stream, src, T, heads, stride, col0, n, (bf16*)dst, gate, gate_ld, gate_elem);
     else
         return SHARPI_BAD_ARGUMENT;
     return SHARPI_OK;

@@ -11,6 +11,8 @@
 //                 with `n_groups` > 1 the experts form equal groups of neighbours, a group's score is its largest choice
 //                 score, and only experts of the `keep` best groups may be chosen (the lowest index among equal groups).
 //                 Weights as for the sigmoid (scale * s / (sum + 1e-20) when `renormalize`).
+//                 `scoring` = 3: s = sigmoid(z) with the groups of 2.  `group_top` = 2: a group's score is the sum of its two
+//                 largest choice scores (of its only one in groups of one) in place of the largest.
 //                 `gate_w` [H] (optional): one more row, gate_out[t] = sigmoid(gate_w . h_t), the gate of a shared expert.
 //   pair_tokens   after the (row, choice) pairs have been sorted by expert: the row each sorted pair belongs to.
 //   combine       out[t] = add[t] + sum over the row's k pairs of y[pair], in the order of the choices.
@@ -33,7 +35,7 @@ __global__ void __launch_bounds__(1024)
 router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                    int T, int H, int E, int k, float scale, int renormalize, int* __restrict__ expert_id,
                    float* __restrict__ weight, float* __restrict__ scores_out, int stage_rows,
-                   const float* __restrict__ bias, int scoring, int n_groups, int keep, const float* __restrict__ gate_w,
+                   const float* __restrict__ bias, int scoring, int n_groups, int keep, int group_top, const float* __restrict__ gate_w,
                    float* __restrict__ gate_out, int vec) {
     extern __shared__ __align__(16) float smem[];         // the rows [ROWS][H] if they fit; per row s [E], choice [E]; group scores
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
@@ -91,7 +93,7 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
             const float z = warp_sum((acc[r][0] + acc[r][1]) + (acc[r][2] + acc[r][3])) + (bias && e < E ? bias[e] : 0.0f);
             if (lane == 0 && r < rows && e == E) gate_out[t0 + r] = 1.0f / (1.0f + expf(-z));
             if (lane == 0 && r < rows && e < E) {
-                const float s = scoring >= 1 ? z : 1.0f / (1.0f + expf(-z));
+                const float s = scoring == 1 || scoring == 2 ? z : 1.0f / (1.0f + expf(-z));
                 score_s[(size_t)r * 2 * E + e] = s;
                 score_s[(size_t)r * 2 * E + E + e] = correction ? s + correction[e] : s;
                 if (scores_out && scoring != 2) scores_out[(size_t)(t0 + r) * E + e] = s;
@@ -120,13 +122,19 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
             if (scores_out) scores_out[(size_t)t * E + e] = s;
         }
         __syncwarp();
+    }
+    if (scoring >= 2) {
         if (n_groups > 1 && keep < n_groups) {
-            float* g_s = score_s + (size_t)TOPK_ROWS * 2 * E + (size_t)warp * n_groups;       // a group's largest choice score
+            float* g_s = score_s + (size_t)TOPK_ROWS * 2 * E + (size_t)warp * n_groups;       // the groups' scores
             const int per = E / n_groups;
             for (int g = lane; g < n_groups; g += 32) {
-                float best = -INFINITY;
-                for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, c_s[e]);
-                g_s[g] = best;
+                float best = -INFINITY, second = -INFINITY;
+                for (int e = g * per; e < (g + 1) * per; ++e) {
+                    const float c = c_s[e];
+                    second = fmaxf(second, fminf(best, c));
+                    best = fmaxf(best, c);
+                }
+                g_s[g] = group_top == 2 && per > 1 ? best + second : best;
             }
             __syncwarp();
             // a group stays when fewer than `keep` groups are ahead of it (larger score, or equal and lower index)
@@ -178,8 +186,8 @@ router_topk_kernel(const float* __restrict__ h, const float* __restrict__ wr, co
 
 static int router_topk_impl(const float* h, const float* wr, const float* correction, int T, int H, int E, int k,
                             float scale, int renormalize, int* expert_id, float* weight, float* scores_out,
-                            const float* bias, int scoring, int n_groups, int keep, const float* gate_w, float* gate_out,
-                            cudaStream_t stream) {
+                            const float* bias, int scoring, int n_groups, int keep, int group_top, const float* gate_w,
+                            float* gate_out, cudaStream_t stream) {
     if (T <= 0) return SHARPI_OK;
     if (H <= 0 || E <= 0 || k <= 0 || k > E || k > 32) return SHARPI_BAD_ARGUMENT;
     const int per_cta = T > TOPK_MANY_ROWS ? 4 : 1;
@@ -196,11 +204,11 @@ static int router_topk_impl(const float* h, const float* wr, const float* correc
     if (per_cta == 4)
         router_topk_kernel<4><<<(T + 3) / 4, warps * 32, smem, stream>>>(
             h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring,
-            n_groups, keep, gate_w, gate_out, vec);
+            n_groups, keep, group_top, gate_w, gate_out, vec);
     else
         router_topk_kernel<1><<<T, warps * 32, smem, stream>>>(
             h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, stage_rows, bias, scoring,
-            n_groups, keep, gate_w, gate_out, vec);
+            n_groups, keep, group_top, gate_w, gate_out, vec);
     SHARPI_CHECK_LAUNCH();
     return SHARPI_OK;
 }
@@ -210,19 +218,20 @@ SHARPI_API int sharpi_router_topk(const float* h, const float* wr, const float* 
                                   const float* bias, int scoring, cudaStream_t stream) {
     if (scoring != 0 && scoring != 1) return SHARPI_BAD_ARGUMENT;
     return router_topk_impl(h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, bias, scoring,
-                            0, 0, nullptr, nullptr, stream);
+                            0, 0, 1, nullptr, nullptr, stream);
 }
 
-// The softmax over all experts, with groups (n_groups >= 1, keep of them; k must fit the kept groups' experts) and the gate row
+// The softmax over all experts (`scoring` 2) or the sigmoid of each (3), with groups (n_groups >= 1, keep of them; k must fit
+// the kept groups' experts) whose score is the sum of their `group_top` largest choice scores, and the gate row
 SHARPI_API int sharpi_router_groups(const float* h, const float* wr, const float* correction, int T, int H, int E, int k,
-                                    float scale, int renormalize, int n_groups, int keep, const float* gate_w,
-                                    float* gate_out, int* expert_id, float* weight, float* scores_out,
+                                    float scale, int renormalize, int n_groups, int keep, int scoring, int group_top,
+                                    const float* gate_w, float* gate_out, int* expert_id, float* weight, float* scores_out,
                                     cudaStream_t stream) {
     if (n_groups < 1 || E % n_groups != 0 || keep < 1 || keep > n_groups || k > keep * (E / n_groups) ||
-        (gate_w == nullptr) != (gate_out == nullptr))
+        (scoring != 2 && scoring != 3) || (group_top != 1 && group_top != 2) || (gate_w == nullptr) != (gate_out == nullptr))
         return SHARPI_BAD_ARGUMENT;
-    return router_topk_impl(h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, nullptr, 2,
-                            n_groups, keep, gate_w, gate_out, stream);
+    return router_topk_impl(h, wr, correction, T, H, E, k, scale, renormalize, expert_id, weight, scores_out, nullptr,
+                            scoring, n_groups, keep, group_top, gate_w, gate_out, stream);
 }
 
 __global__ void pair_tokens_kernel(const int* __restrict__ sorted_pairs, int P, int k, int* __restrict__ tokens) {

@@ -112,7 +112,8 @@ class Engine:
                                   device=self.device, model_state_specs=getattr(self.model, "state_specs", None))
         self.runner = StepRunner(self.model, self.cache)
         self.runner.use_graphs = self.runner.use_graphs and o.cuda_graphs
-        self.scheduler = Scheduler(self.cache, max_batch=o.max_batch, max_tokens_per_step=o.max_tokens_per_step)
+        self.scheduler = Scheduler(self.cache, max_batch=o.max_batch, max_tokens_per_step=o.max_tokens_per_step,
+                                   max_positions=getattr(self.model, "max_positions", None))
         self.sampler = Sampler(self.device)
         self._start_bookkeeping()
 
@@ -126,7 +127,8 @@ class Engine:
         self.device, self.dtype = getattr(cache, "device", None), getattr(model, "act_dtype", None)
         self.model, self.cache, self.runner, self.sampler = model, cache, runner, sampler
         self.scheduler = Scheduler(cache, max_batch=self.options.max_batch,
-                                   max_tokens_per_step=self.options.max_tokens_per_step)
+                                   max_tokens_per_step=self.options.max_tokens_per_step,
+                                   max_positions=getattr(model, "max_positions", None))
         self._start_bookkeeping()
         return self
 
@@ -175,6 +177,9 @@ class Engine:
         for t in prompt:
             if not (0 <= t < V):
                 raise ValueError(f"prompt token {t} is outside the vocabulary [0, {V})")
+        limit = getattr(self.model, "max_positions", None)
+        if limit is not None and len(prompt) > limit:
+            raise ValueError(f"the prompt has {len(prompt)} tokens, the model {limit} positions")
         req = Request(rid, prompt, params, stop_set=params.resolve_stop_set(self.model.eos_token_ids),
                       sampler=SamplerState.start(params, prompt))
         self.scheduler.add(req)

@@ -101,12 +101,15 @@ class StepPlan:
 
 
 class Scheduler:
-    def __init__(self, cache: CacheManager, *, max_batch: int, max_tokens_per_step: int):
+    def __init__(self, cache: CacheManager, *, max_batch: int, max_tokens_per_step: int, max_positions: Optional[int] = None):
+        """``max_positions``: the most positions a sequence may have; a request that reached it ends with ``length`` (its
+        last token is sampled, not run)."""
         if max_batch <= 0 or max_tokens_per_step <= 0:
             raise ValueError("max_batch and max_tokens_per_step must be positive")
         self.cache = cache
         self.max_batch = min(max_batch, cache.max_requests)
         self.max_tokens_per_step = max_tokens_per_step
+        self.max_positions = max_positions
         self.waiting: Deque[Request] = deque()
         self.running: List[Request] = []            # in admission order
         self._order = itertools.count()
@@ -307,7 +310,8 @@ class Scheduler:
                 finished.append(req)
                 continue
             req.generated.append(token)
-            if len(req.generated) >= req.params.max_new_tokens:
+            if len(req.generated) >= req.params.max_new_tokens or (
+                    self.max_positions is not None and len(req.prompt) + len(req.generated) > self.max_positions):
                 self._finish(req, "length")
                 finished.append(req)
         return finished

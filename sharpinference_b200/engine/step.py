@@ -118,6 +118,7 @@ class StepRunner:
         if not entries:
             raise StepError("a step needs at least one entry")
         V = self.model.vocab_size
+        limit = getattr(self.model, "max_positions", None)
         seen = set()
         for e in entries:
             if e.request_id in seen:
@@ -128,6 +129,9 @@ class StepRunner:
             n = len(e.tokens)
             if n == 0:
                 raise StepError(f"request {e.request_id!r}: an entry must bring at least one token", e.request_id)
+            if limit is not None and self.cache.requests[e.request_id].length + n > limit:
+                raise StepError(f"request {e.request_id!r}: position {self.cache.requests[e.request_id].length + n - 1} is beyond "
+                                f"the model's {limit} positions", e.request_id)
             for w in e.want:
                 if not (0 <= w < n):
                     raise StepError(f"request {e.request_id!r}: wanted place {w} is outside its {n} token(s)",

@@ -79,7 +79,7 @@ SIGNATURES: Dict[str, Tuple[str, list]] = {
     "sharpi_add_dyt": ("elementwise", [P, P, P, P, P, P, I, I, P, I, P, P]),
     "sharpi_latent_down_post": ("latent", [P, I, I, I, I, I, P, P, F, P, P, P, I, I, P, P, P, I, I, I, I, I, F, P]),
     "sharpi_head_major": ("latent", [P, I, I, I, I, I, I, P, I, I, P]),
-    "sharpi_head_minor": ("latent", [P, I, I, I, I, I, P, I, P, I, P]),
+    "sharpi_head_minor": ("latent", [P, I, I, I, I, I, P, I, P, I, I, P]),
     "sharpi_latent_q_join": ("latent", [P, P, P, P, I, I, I, I, I, I, I, P, I, I, F, P]),
     "sharpi_ssd_scan": ("mamba2", [P, I, I, I, I, P, I, I, P, P, P, P, P, P, LL, P, I, I, I, I, I, I, P]),
     "sharpi_add_layernorm": ("elementwise", [P, P, P, P, F, P, I, I, P, I, P, P]),
@@ -92,9 +92,16 @@ SIGNATURES: Dict[str, Tuple[str, list]] = {
     "sharpi_lightning_walk": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, LL, P, I, I, I, I, P]),
     "sharpi_lightning_chunks": ("lightning", [P, I, I, I, I, P, P, P, P, I, P, I, P, P, LL, P, I, I, I, I, P]),
     "sharpi_norm_sigmoid_gate": ("lightning", [P, P, I, P, F, F, I, I, P, I, I, P]),
-    "sharpi_router_groups": ("moe_topk", [P, P, P, I, I, I, I, F, I, I, I, P, P, P, P, P, P]),
+    "sharpi_router_groups": ("moe_topk", [P, P, P, I, I, I, I, F, I, I, I, I, I, P, P, P, P, P, P]),
     "sharpi_moe_combine_full": ("moe_topk", [P, P, P, P, P, P, P, P, I, I, I, I, P]),
     "sharpi_tc_grouped_gemm_clamped": ("tc_gemm", [P, P, P, P, P, P, P, I, I, I, I, I, I, F, P]),
+    "sharpi_add_normed": ("sandwich", [P, P, P, P, F, P, I, I, P, I, P, P]),
+    "sharpi_embed_pos": ("sandwich", [P, P, P, P, I, F, P, I, I, I, I, P]),
+    "sharpi_side_gate": ("sandwich", [P, I, P, P, I, LL, I, I, I, P, I, I, I, P]),
+    "sharpi_delta_prep": ("delta", [P, I, P, P, LL, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P]),
+    "sharpi_delta_walk": ("delta", [P, P, P, I, P, P, P, P, P, I, P, LL, P, I, I, I, I, P]),
+    "sharpi_delta_chunks": ("delta", [P, P, P, I, P, P, P, P, P, I, P, I, P, P, P, P, LL, P, I, I, I, I, P]),
+    "sharpi_head_norm_gate": ("delta", [P, P, I, P, F, I, I, I, P, I, P]),
     "sharpi_gated_group_norm": ("mamba2", [P, P, I, P, F, I, I, I, P, I, P]),
 }
 

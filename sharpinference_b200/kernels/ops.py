@@ -1300,7 +1300,7 @@ def add_dyt(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor
 
 
 def latent_down_post(down: torch.Tensor, *, q_rank: int, rank: int, rot: int, rot_dims: int,
-                     q_norm_weight: Optional[torch.Tensor], c_norm_weight: torch.Tensor, eps: float,
+                     q_norm_weight: Optional[torch.Tensor], c_norm_weight: Optional[torch.Tensor], eps: float,
                      positions: torch.Tensor, row_req: torch.Tensor, block_table: torch.Tensor,
                      inv_freq: Optional[torch.Tensor], kv_layer: torch.Tensor, page_size: int,
                      write_kv: bool = True, rot_amplitude: float = 1.0) -> torch.Tensor:
@@ -1308,13 +1308,15 @@ def latent_down_post(down: torch.Tensor, *, q_rank: int, rank: int, rot: int, ro
     query latent ``[T, q_rank]`` in the cache's dtype (returned), and ``[c | k_rot | 0]`` written into every row's
     place in ``kv_layer [pages, planes, 1, page_size, D]`` (``[c | 0]`` into the value plane when there are two).
     ``down`` may be a column range of a wider product (rows apart); ``rot_amplitude`` multiplies the rotation's
-    cosines and sines."""
+    cosines and sines.  Without ``write_kv`` only the query latent is normed: ``down`` is ``[T, q_rank]`` and there is no
+    ``c_norm_weight``."""
     ld = _need_columns(down, "down", torch.float32)
-    _need(c_norm_weight, "c_norm_weight", torch.float32)
+    if write_kv:
+        _need(c_norm_weight, "c_norm_weight", torch.float32)
     _need(kv_layer, "kv_layer")
     T = down.shape[0]
     planes, D = int(kv_layer.shape[1]), int(kv_layer.shape[-1])
-    if tuple(kv_layer.shape[1:]) != (planes, 1, page_size, D) or down.shape[1] != q_rank + rank + rot:
+    if tuple(kv_layer.shape[1:]) != (planes, 1, page_size, D) or down.shape[1] != q_rank + (rank + rot if write_kv else 0):
         raise KernelError(f"kv_layer {tuple(kv_layer.shape)} or the projection's width {ld} disagree with the sizes")
     if inv_freq is not None:
         _need(inv_freq, "inv_freq", torch.float32)
@@ -1322,7 +1324,7 @@ def latent_down_post(down: torch.Tensor, *, q_rank: int, rank: int, rot: int, ro
             raise KernelError(f"{rot_dims} rotated elements need {rot_dims // 2} frequencies, found {inv_freq.numel()}")
     cq = torch.empty((T, q_rank), dtype=kv_layer.dtype, device=down.device)
     check(kernel("sharpi_latent_down_post")(down.data_ptr(), ld, q_rank, rank, rot, rot_dims if inv_freq is not None else 0,
-                                            _ptr(q_norm_weight), c_norm_weight.data_ptr(), float(eps), positions.data_ptr(),
+                                            _ptr(q_norm_weight), _ptr(c_norm_weight), float(eps), positions.data_ptr(),
                                             row_req.data_ptr(), block_table.data_ptr(), block_table.shape[-1], page_size,
                                             _ptr(inv_freq), cq.data_ptr(), kv_layer.data_ptr(), planes, D, int(write_kv),
                                             dtype_code(kv_layer.dtype), T, float(rot_amplitude), _stream()),
@@ -1347,18 +1349,19 @@ def head_major(src: torch.Tensor, *, heads: int, stride: int, col0: int, n: int,
 def head_minor(src: torch.Tensor, *, heads: int, out_dtype: torch.dtype, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``src`` float32 ``[heads * T, n]`` (head by head) as ``[T, heads * n]`` in ``out_dtype``.  ``gate`` float32
     ``[T, heads]`` (possibly a column range of a wider product): head ``h`` of row ``t`` is multiplied by
-    ``sigmoid(gate[t, h])``."""
+    ``sigmoid(gate[t, h])``; ``[T, heads * n]``: every element by its own."""
     _need(src, "src", torch.float32)
     n = src.shape[1]
     T = src.shape[0] // heads
-    gate_ld = 0
+    gate_ld = elem = 0
     if gate is not None:
         gate_ld = _need_columns(gate, "gate", torch.float32)
-        if tuple(gate.shape) != (T, heads):
-            raise KernelError(f"gate is {tuple(gate.shape)}, expected [{T}, {heads}]")
+        if tuple(gate.shape) not in ((T, heads), (T, heads * n)):
+            raise KernelError(f"gate is {tuple(gate.shape)}, expected [{T}, {heads}] or [{T}, {heads * n}]")
+        elem = int(gate.shape[1] == heads * n)
     out = torch.empty((T, heads * n), dtype=out_dtype, device=src.device)
     check(kernel("sharpi_head_minor")(src.data_ptr(), T, heads, n, 0, n, out.data_ptr(), dtype_code(out_dtype),
-                                      _ptr(gate), gate_ld, _stream()), "sharpi_head_minor")
+                                      _ptr(gate), gate_ld, elem, _stream()), "sharpi_head_minor")
     return out
 
 
@@ -1687,11 +1690,16 @@ def norm_sigmoid_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor,
 # ---------------------------------------------------------------------------------------
 # mixtures routed by a softmax over all experts, in groups, with identity experts
 # ---------------------------------------------------------------------------------------
+GROUP_ROUTER_SCORING = {"softmax": 2, "sigmoid": 3}
+
+
 def router_groups(h32: torch.Tensor, router_weight: torch.Tensor, k: int, *, correction: Optional[torch.Tensor] = None,
                   scale: float = 1.0, renormalize: bool = True, n_groups: int = 1, keep: int = 1,
-                  gate_weight: Optional[torch.Tensor] = None, want_scores: bool = False):
-    """``s = softmax(h . Wr^T)`` in float32; the ``k`` largest of ``s + correction`` among the experts of the ``keep`` best of
-    ``n_groups`` groups of neighbours (a group's score is its largest ``s + correction``); weights ``scale * s``, divided by
+                  gate_weight: Optional[torch.Tensor] = None, want_scores: bool = False, scoring: str = "softmax",
+                  group_top: int = 1):
+    """``s = softmax(h . Wr^T)`` (or ``sigmoid``: ``scoring``) in float32; the ``k`` largest of ``s + correction`` among the experts of the ``keep`` best of
+    ``n_groups`` groups of neighbours (a group's score is its largest ``s + correction``, or with ``group_top`` = 2 the sum of
+    its two largest); weights ``scale * s``, divided by
     the chosen ``s``' sum + 1e-20 first when ``renormalize``.  ``gate_weight`` float32 ``[H]``: also
     ``sigmoid(gate_weight . h)`` per row.  Returns ``(expert int32 [T, k], weight float32 [T, k], gate [T] or None, scores
     [T, E] or None)``."""
@@ -1707,6 +1715,8 @@ def router_groups(h32: torch.Tensor, router_weight: torch.Tensor, k: int, *, cor
             raise KernelError(f"correction has {correction.numel()} entries for {E} experts")
     if n_groups < 1 or E % n_groups or not (1 <= keep <= n_groups) or not (1 <= k <= min(keep * (E // n_groups), 32)):
         raise KernelError(f"{k} of {E} experts in {n_groups} groups of which {keep} are kept")
+    if scoring not in GROUP_ROUTER_SCORING or group_top not in (1, 2):
+        raise KernelError(f"scoring '{scoring}' must be softmax or sigmoid and group_top ({group_top}) 1 or 2")
     if gate_weight is not None:
         _need(gate_weight, "gate_weight", torch.float32)
         if gate_weight.numel() != H:
@@ -1716,8 +1726,8 @@ def router_groups(h32: torch.Tensor, router_weight: torch.Tensor, k: int, *, cor
     gate = torch.empty((T,), dtype=torch.float32, device=h32.device) if gate_weight is not None else None
     scores = torch.empty((T, E), dtype=torch.float32, device=h32.device) if want_scores else None
     check(kernel("sharpi_router_groups")(h32.data_ptr(), router_weight.data_ptr(), _ptr(correction), T, H, E, k,
-                                         float(scale), int(renormalize), int(n_groups), int(keep), _ptr(gate_weight),
-                                         _ptr(gate), expert.data_ptr(), weight.data_ptr(), _ptr(scores), _stream()),
+                                         float(scale), int(renormalize), int(n_groups), int(keep), GROUP_ROUTER_SCORING[scoring],
+                                         int(group_top), _ptr(gate_weight), _ptr(gate), expert.data_ptr(), weight.data_ptr(), _ptr(scores), _stream()),
           "sharpi_router_groups")
     return expert, weight, gate, scores
 
@@ -1770,4 +1780,163 @@ def tc_grouped_gemm_clamped(a: torch.Tensor, w: torch.Tensor, group_offsets: tor
                                                    status_word(a.device).data_ptr(), _ptr(partial), _ptr(tickets), rows, N, K,
                                                    E, row_tile, k_split, float(limit), _stream()),
           "sharpi_tc_grouped_gemm_clamped")
+    return out
+
+
+# ---------------------------------------------------------------------------------------
+# sublayer outputs that are normed before they enter the stream; learned positions; a token's own vector (sandwich.cu)
+# ---------------------------------------------------------------------------------------
+def add_normed(x: torch.Tensor, y: torch.Tensor, y_weight: torch.Tensor, weight: Optional[torch.Tensor], eps: float,
+               out_dtype: torch.dtype, *, rows: Optional[torch.Tensor] = None, want_fp32: bool = False):
+    """``x += y / sqrt(mean(y^2) + eps) * y_weight`` in place, and the RMS norm of the new ``x`` under ``weight`` (``x`` itself
+    in ``out_dtype`` when ``weight`` is None) for every row.  With ``rows`` (int32 indices) only those rows are formed and
+    ``x`` stays as it is.  Returns ``(out, out32)`` as :func:`add_rmsnorm` does."""
+    for name, t in (("x", x), ("y", y), ("y_weight", y_weight)) + ((("weight", weight),) if weight is not None else ()):
+        _need(t, name, torch.float32)
+    H = x.shape[-1]
+    if y.shape != x.shape or y_weight.numel() != H or (weight is not None and weight.numel() != H):
+        raise KernelError(f"x {tuple(x.shape)}, y {tuple(y.shape)} and the weights disagree")
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    T = rows.numel() if rows is not None else x.numel() // H
+    out = torch.empty((T, H), dtype=out_dtype, device=x.device)
+    out32 = None
+    if want_fp32:
+        out32 = out if out_dtype == torch.float32 else torch.empty((T, H), dtype=torch.float32, device=x.device)
+    check(kernel("sharpi_add_normed")(x.data_ptr(), y.data_ptr(), y_weight.data_ptr(), _ptr(weight), float(eps), _ptr(rows), T, H,
+                                      out.data_ptr(), dtype_code(out_dtype), None if out32 is out else _ptr(out32), _stream()),
+          "sharpi_add_normed")
+    return out, out32
+
+
+def embed_pos(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos: torch.Tensor, scale: float) -> torch.Tensor:
+    """``table[ids[t]] * scale + pos[positions[t]]`` as float32."""
+    _need(ids, "ids", torch.int32)
+    _need(positions, "positions", torch.int32)
+    _need(table, "table")
+    _need(pos, "pos", table.dtype)
+    T, (V, H) = ids.numel(), table.shape
+    if pos.shape[1] != H or positions.numel() != T:
+        raise KernelError(f"the position table is {tuple(pos.shape)}, the embedding {tuple(table.shape)}")
+    out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    check(kernel("sharpi_embed_pos")(ids.data_ptr(), positions.data_ptr(), table.data_ptr(), pos.data_ptr(), dtype_code(table.dtype),
+                                     float(scale), out.data_ptr(), T, H, V, pos.shape[0], _stream()), "sharpi_embed_pos")
+    return out
+
+
+def side_gate(gate: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col0: int, n: int, out_dtype: torch.dtype) -> torch.Tensor:
+    """``gelu_tanh(gate[t, j]) * table[ids[t], col0 + j]`` for the first ``n`` columns of ``gate`` (float32 ``[T, n_out]``), zeros
+    in the others."""
+    ld = _need_columns(gate, "gate", torch.float32)
+    _need(ids, "ids", torch.int32)
+    _need(table, "table")
+    T, n_out = gate.shape
+    if n > n_out or col0 + n > table.shape[1] or ids.numel() != T:
+        raise KernelError(f"columns {col0} .. {col0 + n} of a table {tuple(table.shape)} behind a gate {tuple(gate.shape)}")
+    out = torch.empty((T, n_out), dtype=out_dtype, device=gate.device)
+    check(kernel("sharpi_side_gate")(gate.data_ptr(), ld, ids.data_ptr(), table.data_ptr(), dtype_code(table.dtype), table.shape[1],
+                                     int(col0), int(n), n_out, out.data_ptr(), dtype_code(out_dtype), T, table.shape[0], _stream()),
+          "sharpi_side_gate")
+    return out
+
+
+# ---------------------------------------------------------------------------------------
+# the gated delta rule with a decay per key channel (delta.cu)
+# ---------------------------------------------------------------------------------------
+DELTA_CHUNK = 16             # rows of a chunk
+DELTA_MAX_KEY = 512          # key size the walk takes
+DELTA_MAX_CHUNK_KEY = 256    # key size up to which long portions are cut into chunks
+
+
+def delta_state_floats(heads: int, d: int, dv: int) -> int:
+    """Floats of a request's state: a column per value element, of ``d`` rounded up to a multiple of 4."""
+    return heads * dv * ((d + 3) // 4 * 4)
+
+
+def delta_prep(proj: torch.Tensor, *, conv_weight: torch.Tensor, conv_state: Optional[torch.Tensor], row_offsets: torch.Tensor,
+               state_slots: torch.Tensor, tiles: Optional[torch.Tensor], kv_heads: int, heads: int, d: int, dv: int, low: int,
+               act_dtype: torch.dtype):
+    """Behind the fused projection ``proj`` float32 ``[T, q | k | v | low | b | ...]``: ``(qkv, beta, low)`` with ``qkv`` float32
+    ``[T, channels]`` (convolved under ``conv_weight [taps, channels]``, silu, q and k unit vectors per head, q times
+    d^(-1/2)), ``beta = sigmoid(b)`` float32 ``[T, heads]`` and the ``low`` columns in ``act_dtype``.  ``conv_state``
+    ``[slots, (taps - 1) * channels]`` is moved on.  ``tiles`` int32 ``[n, 4]``: pieces of requests' rows (None: a request a
+    piece)."""
+    ld = _need_columns(proj, "proj", torch.float32)
+    _need(conv_weight, "conv_weight", torch.float32)
+    _need(row_offsets, "row_offsets", torch.int32)
+    _need(state_slots, "state_slots", torch.int32)
+    T, (taps, channels) = proj.shape[0], conv_weight.shape
+    if channels != 2 * kv_heads * d + heads * dv or channels + low + heads > proj.shape[1]:
+        raise KernelError(f"{channels} channels and a projection of {proj.shape[1]} columns disagree with the sizes")
+    if taps > 1:
+        _need(conv_state, "conv_state", torch.float32)
+        if conv_state.shape[-1] != (taps - 1) * channels:
+            raise KernelError(f"the convolution's state holds {conv_state.shape[-1]} floats, expected {(taps - 1) * channels}")
+    if tiles is not None:
+        _need(tiles, "tiles", torch.int32)
+    qkv = torch.empty((T, channels), dtype=torch.float32, device=proj.device)
+    beta = torch.empty((T, heads), dtype=torch.float32, device=proj.device)
+    out = torch.empty((T, low), dtype=act_dtype, device=proj.device)
+    check(kernel("sharpi_delta_prep")(proj.data_ptr(), ld, conv_weight.data_ptr(), _ptr(conv_state) if taps > 1 else None,
+                                      conv_state.stride(0) if taps > 1 else 0, row_offsets.data_ptr(), state_slots.data_ptr(),
+                                      _ptr(tiles), tiles.shape[0] if tiles is not None else state_slots.numel(), qkv.data_ptr(),
+                                      beta.data_ptr(), out.data_ptr(), dtype_code(act_dtype), kv_heads, heads, d, dv, taps, low,
+                                      float(d) ** -0.5, _stream()), "sharpi_delta_prep")
+    return qkv, beta, out
+
+
+def delta_rule(qkv: torch.Tensor, beta: torch.Tensor, z: torch.Tensor, *, dt_bias: torch.Tensor, a_log: torch.Tensor,
+               row_offsets: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, kv_heads: int, heads: int, d: int,
+               dv: int, num_requests: int, walk_requests: Optional[torch.Tensor] = None, num_walk: Optional[int] = None,
+               chunks: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q`` per head, ``g = exp(-exp(a_log) softplus(z + dt_bias))`` per
+    key channel: float32 ``[T, heads * dv]``.  ``qkv`` and ``beta`` as :func:`delta_prep` leaves them, ``z`` float32
+    ``[T, heads * d]`` (possibly a column range), ``state`` ``[slots, delta_state_floats]``.  ``walk_requests`` (None: all) are
+    walked row by row, the requests of ``spans`` (int32 ``[m, 4]``) by chunks (int32 ``[n, 4]``, at most DELTA_CHUNK rows)."""
+    ldz = _need_columns(z, "z", torch.float32)
+    for name, t in (("qkv", qkv), ("beta", beta), ("dt_bias", dt_bias), ("a_log", a_log), ("state", state)):
+        _need(t, name, torch.float32)
+    _need(row_offsets, "row_offsets", torch.int32)
+    _need(state_slots, "state_slots", torch.int32)
+    T = qkv.shape[0]
+    if (qkv.shape[1] != 2 * kv_heads * d + heads * dv or tuple(beta.shape) != (T, heads) or tuple(z.shape) != (T, heads * d)
+            or dt_bias.numel() != heads * d or a_log.numel() != heads):
+        raise KernelError("the delta rule's operands disagree with the sizes")
+    if state[0].numel() != delta_state_floats(heads, d, dv):
+        raise KernelError(f"state rows hold {state[0].numel()} floats, expected {delta_state_floats(heads, d, dv)}")
+    y = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
+    n_walk = num_requests if num_walk is None else int(num_walk)
+    common = (qkv.data_ptr(), beta.data_ptr(), z.data_ptr(), ldz, dt_bias.data_ptr(), a_log.data_ptr(), row_offsets.data_ptr(),
+              state_slots.data_ptr())
+    if chunks is not None:
+        _need(chunks, "chunks", torch.int32)
+        _need(spans, "spans", torch.int32)
+        n, dp = chunks.shape[0], (d + 3) // 4 * 4
+        mats = torch.empty((n * heads * dp, 3 * DELTA_CHUNK), dtype=torch.float32, device=qkv.device)
+        last = torch.empty((n * heads, dp), dtype=torch.float32, device=qkv.device)
+        u0 = torch.empty((n * heads * DELTA_CHUNK, dv), dtype=torch.float32, device=qkv.device)
+        check(kernel("sharpi_delta_chunks")(*common, chunks.data_ptr(), n, spans.data_ptr(), spans.shape[0], mats.data_ptr(),
+                                            last.data_ptr(), u0.data_ptr(), state.data_ptr(), state.stride(0), y.data_ptr(),
+                                            kv_heads, heads, d, dv, _stream()), "sharpi_delta_chunks")
+    if n_walk:
+        if walk_requests is not None:
+            _need(walk_requests, "walk_requests", torch.int32)
+        check(kernel("sharpi_delta_walk")(*common, _ptr(walk_requests), n_walk, state.data_ptr(), state.stride(0), y.data_ptr(),
+                                          kv_heads, heads, d, dv, _stream()), "sharpi_delta_walk")
+    return y
+
+
+def head_norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, heads: int,
+                   out_dtype: torch.dtype) -> torch.Tensor:
+    """Every head of ``y`` float32 ``[T, heads * dv]`` divided by its root mean square, times ``weight [dv]`` (shared by the
+    heads) and ``sigmoid(gate)`` (float32 ``[T, heads * dv]``, possibly a column range)."""
+    _need(y, "y", torch.float32)
+    _need(weight, "weight", torch.float32)
+    ld = _need_columns(gate, "gate", torch.float32)
+    T, n = y.shape
+    if tuple(gate.shape) != (T, n) or weight.numel() * heads != n:
+        raise KernelError(f"y {tuple(y.shape)}, gate {tuple(gate.shape)} and weight {weight.numel()} disagree for {heads} heads")
+    out = torch.empty((T, n), dtype=out_dtype, device=y.device)
+    check(kernel("sharpi_head_norm_gate")(y.data_ptr(), gate.data_ptr(), ld, weight.data_ptr(), float(eps), T, heads, n // heads,
+                                          out.data_ptr(), dtype_code(out_dtype), _stream()), "sharpi_head_norm_gate")
     return out

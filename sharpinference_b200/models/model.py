@@ -48,6 +48,8 @@ class DecoderModel:
         self.config = config
         self.embedder = embedder
         self.state_specs = dict(getattr(embedder, "state_specs", None) or {})
+        # most positions a sequence may have (None: as many as the cache holds); a table of learned positions sets it
+        self.max_positions: Optional[int] = getattr(embedder, "max_positions", None)
         self.logit_scale = float(logit_scale)
         self.embedding_scale = float(embedding_scale)
         self.logit_softcap = float(logit_softcap)

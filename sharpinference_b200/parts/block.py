@@ -14,6 +14,11 @@ as ``pending`` and the next block's first norm (or the model's last) adds it.  A
 ``eps`` are one kernel.  Where the mixer and the feed-forward both end in a plain product (a :class:`ColumnMixer` beside a
 feed-forward with ``out_columns``), their inner columns lie side by side in one matrix and one product forms the sum of
 both outputs.
+
+``SandwichBlock`` norms what a sublayer returns as well: ``x += scale1 * post1(mixer(norm1(x)))``, ``x += scale2 *
+post2(ffn(norm2(x)))``, and may end with a token's own vector through a gate that reads the stream (:class:`TokenSide`).
+All updates are :class:`NormedUpdate`: one kernel norms a sublayer's output, adds it and norms the stream for whatever
+reads it next.
 """
 from __future__ import annotations
 
@@ -25,8 +30,9 @@ from ..kernels import ops
 from .base import Block, ColumnMixer, FeedForward, LayerSlot, Mixer, Norm, StepContext, register_part
 from .branches import side_by_side, pad_columns
 from .linear import Linear
-from .norm import RMSNorm
+from .norm import NormedUpdate, RMSNorm
 from .side import fork, join
+from .token_side import TokenSide
 
 
 @register_part("block", "prenorm")
@@ -106,3 +112,38 @@ class ParallelPairBlock(Block):
         y = self.ffn.forward(ctx, h2, h32)
         join(side)
         return x, ops.add(mixed, y, out=mixed)
+
+
+@register_part("block", "sandwich")
+class SandwichBlock(Block):
+    """``mixer_post`` / ``ffn_post``: the weights of the norms behind the sublayers; ``mixer_scale`` / ``ffn_scale``: a factor
+    per element of the stream (None: none), formed into the weights once, in float32.  ``side``: the layer's
+    :class:`TokenSide` (None: none)."""
+
+    def __init__(self, *, mixer_norm: RMSNorm, mixer: Mixer, mixer_post: RMSNorm, mixer_scale: Optional[torch.Tensor] = None,
+                 ffn_norm: Optional[RMSNorm] = None, ffn: Optional[FeedForward] = None, ffn_post: Optional[RMSNorm] = None,
+                 ffn_scale: Optional[torch.Tensor] = None, side: Optional[TokenSide] = None,
+                 act_dtype: torch.dtype = torch.bfloat16):
+        if (ffn is None) != (ffn_norm is None) or (ffn is None) != (ffn_post is None):
+            raise ValueError("a feed-forward comes with the norms before and behind it, and only then")
+        self.mixer_norm, self.mixer, self.ffn_norm, self.ffn, self.side = mixer_norm, mixer, ffn_norm, ffn, side
+        self.act_dtype = act_dtype
+
+        def scaled(norm: RMSNorm, scale):
+            return norm.weight if scale is None else (norm.weight * scale.to(torch.float32)).contiguous()
+        self.mixer_weight, self.mixer_eps = scaled(mixer_post, mixer_scale), mixer_post.eps
+        if ffn is not None:
+            self.ffn_weight, self.ffn_eps = scaled(ffn_post, ffn_scale), ffn_post.eps
+
+    def forward(self, ctx: StepContext, slot: LayerSlot, x: torch.Tensor, pending):
+        h, _ = self.mixer_norm.apply(x, pending, rows=None, out_dtype=self.act_dtype)
+        pending = NormedUpdate(self.mixer.forward(ctx, slot, h), self.mixer_weight, self.mixer_eps)
+        if self.ffn is not None:
+            h, h32 = self.ffn_norm.apply(x, pending, rows=None, out_dtype=self.act_dtype, want_fp32=self.ffn.wants_fp32_input)
+            pending = NormedUpdate(self.ffn.forward(ctx, h, h32), self.ffn_weight, self.ffn_eps)
+        if self.side is not None:
+            pending = self.side.update(ctx, x, pending)
+        return x, pending
+
+    def traced_stream(self, x: torch.Tensor, pending) -> torch.Tensor:
+        return x + pending.value()

@@ -2,7 +2,7 @@
 always-on shared expert, a dense two-layer network with a plain activation (``DenseMLP``) and a
 sigmoid-routed mixture in which every row uses k such networks (``MoESigmoidTopK``), its gated form
 (``MoESigmoidTopKGated``), and a mixture routed by a softmax over all experts in groups, with identity experts, clamped
-gates and a gated shared expert (``MoESoftmaxGroups``).
+gates and a gated shared expert (``MoESoftmaxGroups``), or by a sigmoid of each (``MoESigmoidGroups``).
 
 Dense (src/SharpInference.Engine/ForwardPass.cs:2006-2015): ``y = (silu(h Wg^T) * (h Wu^T)) Wd^T``.
 
@@ -405,6 +405,9 @@ class MoESoftmaxGroups(FeedForward):
     """A mixture of ``E`` gated experts and ``identity`` experts that hand their input on, of which every row uses
     ``top_k``, with an optional shared expert that every row uses.
 
+    The scores may be ``sigmoid(Wr h)`` of each expert instead of the softmax (``scoring``), and a group's score the sum of
+    its two largest choice scores instead of the largest (``group_top = 2``); see :class:`MoESigmoidGroups`.
+
     Router (float32, on the unrounded activations): ``s = softmax(Wr h)`` over all ``E + identity`` experts; choice score
     ``s + correction``; the experts form ``groups`` equal groups of neighbours, only those of the ``keep`` groups with the
     largest choice score in them can be chosen, and of these the ``top_k`` with the largest choice scores are (the lowest
@@ -427,9 +430,13 @@ class MoESoftmaxGroups(FeedForward):
                  identity: int = 0, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
                  route_scale: float = 1.0, renormalize: bool = True, limit: float = 0.0,
                  shared: Optional[DenseSwiGLU] = None, shared_gate: Optional[torch.Tensor] = None,
-                 act_dtype: torch.dtype = torch.bfloat16):
+                 act_dtype: torch.dtype = torch.bfloat16, scoring: str = "softmax", group_top: int = 1):
         E = experts_gate_up.num_groups
         N = E + int(identity)
+        if scoring not in ops.GROUP_ROUTER_SCORING or group_top not in (1, 2):
+            raise ValueError(f"scoring '{scoring}' must be one of {', '.join(ops.GROUP_ROUTER_SCORING)} and group_top "
+                             f"({group_top}) 1 or 2")
+        self.scoring, self.group_top = scoring, int(group_top)
         if identity < 0 or router.shape != (N, experts_gate_up.in_features):
             raise ValueError(f"router weight is {tuple(router.shape)}, expected [{N}, {experts_gate_up.in_features}]")
         if experts_down.num_groups != E or experts_gate_up.out_features != 2 * experts_down.in_features:
@@ -463,7 +470,8 @@ class MoESoftmaxGroups(FeedForward):
                 shared = self.shared.forward(ctx, h)
         expert, weight, gate, _ = ops.router_groups(h32, self.router, k, correction=self.correction, scale=self.route_scale,
                                                     renormalize=self.renormalize, n_groups=self.groups, keep=self.keep,
-                                                    gate_weight=self.shared_gate)
+                                                    gate_weight=self.shared_gate, scoring=self.scoring,
+                                                    group_top=self.group_top)
         if "router_choices" in ctx.extras:          # tracing: which experts every row went to
             ctx.extras["router_choices"].append(expert)
         offsets, sorted_pairs = ops.moe_sort(expert.view(-1), E + self.identity)      # pair = row * k + choice
@@ -491,4 +499,16 @@ class MoESoftmaxGroups(FeedForward):
             join(side)
         if add_ready is not None:
             join(add_ready)
+        if shared is None and self.identity == 0:
+            return ops.moe_combine(y, k, add=add_to, out=add_to)
         return ops.moe_combine_full(y, expert, weight, h32, E, shared=shared, gate=gate, add=add_to, out=add_to)
+
+
+@register_part("feed_forward", "moe_sigmoid_groups")
+class MoESigmoidGroups(MoESoftmaxGroups):
+    """The mixture of :class:`MoESoftmaxGroups` with the other scores: ``s = sigmoid(Wr h)`` of every expert by itself; choice
+    score ``s + correction``; a group's score is the sum of its two largest choice scores; the weights are the chosen ``s``
+    as they are unless ``renormalize``."""
+
+    def __init__(self, *, renormalize: bool = False, group_top: int = 2, **params):
+        super().__init__(renormalize=renormalize, scoring="sigmoid", group_top=group_top, **params)

@@ -22,7 +22,9 @@ product.
 Variants, each a constructor argument: queries that come straight from the input (``q_rank = 0``: ``q = W_q h``, no
 query latent; ``W_q`` then rides in the fused down projection); no rotated part (``rot_dim = 0``); a sliding window
 instead of the whole past (``mask="window"``, ``span``); a gate per head, ``out_h *= sigmoid(W_g h)_h``, whose ``H``
-rows are the last rows of the fused projection (``head_gate``); a rotation whose cosines and sines carry an amplitude
+rows are the last rows of the fused projection (``head_gate``), or a gate per element, ``out *= sigmoid(W_g h)``, with
+``H vdim`` such rows (``element_gate``); a layer without ``W_dkv`` that reads the latents an earlier layer cached through
+its own ``W_uk`` and ``W_uv`` (``borrows``; a schedule entry with ``cache_from``); a rotation whose cosines and sines carry an amplitude
 (``RotaryEncoding(amplitude=...)``, as stretched frequencies bring one).
 """
 from __future__ import annotations
@@ -41,15 +43,16 @@ from .linear import GroupedLinear, Linear
 class LatentAttention(Mixer):
     graph_safe = True
 
-    def __init__(self, *, down: Linear, q_norm_weight: Optional[torch.Tensor], c_norm_weight: torch.Tensor,
+    def __init__(self, *, down: Linear, q_norm_weight: Optional[torch.Tensor], c_norm_weight: Optional[torch.Tensor],
                  up_q: Optional[Linear], up_k: GroupedLinear, up_v: GroupedLinear, out: Linear, num_heads: int, dim: int,
                  rot_dim: int, value_dim: int, q_rank: int, kv_rank: int, eps: float, softmax_scale: float,
                  position: Optional[PositionEncoding] = None, act_dtype: torch.dtype = torch.bfloat16,
-                 mask: str = "full", span: int = 0, head_gate: bool = False):
+                 mask: str = "full", span: int = 0, head_gate: bool = False, element_gate: bool = False, borrows: bool = False):
         """``down``: the fused down projections, rows ``[W_dq (q_rank) | W_dkv (kv_rank + rot_dim)]``; with
         ``q_rank = 0`` (``up_q`` and ``q_norm_weight`` None) the queries themselves lead it:
         ``[W_q (heads * (dim + rot_dim)) | W_dkv (kv_rank + rot_dim)]``; with ``head_gate`` the gate's ``heads`` rows
-        follow.  ``up_k``: per head ``W_uk_h^T`` as a group ``[kv_rank, dim]`` (it maps a head's unrotated query into the
+        follow, with ``element_gate`` its ``heads * value_dim`` rows.  ``borrows``: no ``W_dkv`` rows and no
+        ``c_norm_weight`` (and no rotated part).  ``up_k``: per head ``W_uk_h^T`` as a group ``[kv_rank, dim]`` (it maps a head's unrotated query into the
         latent); ``up_v``: per head ``W_uv_h [value_dim, kv_rank]``.  ``position``: a rotary encoding of neighbouring
         pairs over the first ``rot_dims`` of the ``rot_dim`` rotated elements (None: no rotation).  ``mask``:
         ``"full"`` or ``"window"`` of ``span`` positions, the query's own included."""
@@ -57,10 +60,14 @@ class LatentAttention(Mixer):
         if mask not in ("full", "window") or (mask == "window" and span <= 0):
             raise ValueError(f"mask '{mask}' must be full or a window of a positive span (found {span})")
         lead = q_rank if q_rank > 0 else H * (dim + rot_dim)
-        if down.out_features != lead + kv_rank + rot_dim + (H if head_gate else 0):
-            raise ValueError(f"the fused down projection has {down.out_features} rows, expected "
-                             f"{lead + kv_rank + rot_dim + (H if head_gate else 0)} (queries or their latent {lead}, "
-                             f"key/value latent {kv_rank}, rotated key {rot_dim}, gate {H if head_gate else 0})")
+        if head_gate and element_gate:
+            raise ValueError("the gate is per head or per element, not both")
+        if borrows and (rot_dim or c_norm_weight is not None):
+            raise ValueError("a borrowing layer has no latent of its own: no norm weight for it and no rotated key")
+        tail, gates = 0 if borrows else kv_rank + rot_dim, H if head_gate else H * value_dim if element_gate else 0
+        if down.out_features != lead + tail + gates:
+            raise ValueError(f"the fused down projection has {down.out_features} rows, expected {lead + tail + gates} "
+                             f"(queries or their latent {lead}, key/value latent and rotated key {tail}, gate {gates})")
         if (q_rank > 0) != (up_q is not None) or (q_rank > 0) != (q_norm_weight is not None):
             raise ValueError("a query latent (q_rank > 0) comes with its up projection and norm weight, and only then")
         if up_q is not None and (up_q.in_features != q_rank or up_q.out_features != H * (dim + rot_dim)):
@@ -72,10 +79,12 @@ class LatentAttention(Mixer):
             raise ValueError(f"up_v must hold [{H}, {value_dim}, {kv_rank}]")
         if out.in_features != H * value_dim:
             raise ValueError(f"output projection reads {out.in_features} columns, expected {H * value_dim}")
-        if (q_norm_weight is not None and q_norm_weight.numel() != q_rank) or c_norm_weight.numel() != kv_rank:
+        if (q_norm_weight is not None and q_norm_weight.numel() != q_rank) or (
+                not borrows and c_norm_weight.numel() != kv_rank):
             raise ValueError("the latents' norm weights disagree with q_rank or kv_rank")
         self.inv_freq, self.rot_dims, self.rot_amplitude = None, 0, 1.0
-        self.head_gate, self._lead = bool(head_gate), lead
+        self.head_gate, self.element_gate, self.borrows = bool(head_gate), bool(element_gate), bool(borrows)
+        self._lead, self._tail = lead, tail
         if position is not None and rot_dim:
             self.rot_amplitude = float(getattr(position, "amplitude", 1.0))
             rot = position.rotary()
@@ -107,24 +116,24 @@ class LatentAttention(Mixer):
         table = ctx.block_tables[slot.group]
         mask_kind = ops.MASK_WINDOW if self.cache_spec.kind == "window" else ops.MASK_FULL
         mask_span = max(self.cache_spec.span, 1)
-        down = self.down(h)                                    # [T, (q_rank or H (dim + rot)) + kv_rank + rot (+ H)] float32
-        tail = self.kv_rank + self.rot_dim
-        gate = down[:, self._lead + tail:] if self.head_gate else None
-        if self.q_rank > 0:
-            cq = ops.latent_down_post(down[:, : self._lead + tail], q_rank=self.q_rank, rank=self.kv_rank, rot=self.rot_dim,
+        down = self.down(h)                                    # [T, (q_rank or H (dim + rot)) + kv_rank + rot (+ gate)] float32
+        tail = self._tail
+        gate = down[:, self._lead + tail:] if self.head_gate or self.element_gate else None
+        if self.borrows and slot.writes_cache:
+            raise ValueError("a layer without a latent of its own needs a schedule entry that reads another one's cache")
+        # a layer that reads another one's cache norms its query latent (if it has one) and caches nothing
+        own = tail if slot.writes_cache else 0
+        cq = None
+        if self.q_rank > 0 or own:
+            first = 0 if self.q_rank > 0 else self._lead
+            cq = ops.latent_down_post(down[:, first: self._lead + own], q_rank=self.q_rank, rank=self.kv_rank, rot=self.rot_dim,
                                       rot_dims=self.rot_dims, q_norm_weight=self.q_norm_weight,
                                       c_norm_weight=self.c_norm_weight, eps=self.eps, positions=ctx.positions,
                                       row_req=ctx.row_request, block_table=table, inv_freq=self.inv_freq, kv_layer=slot.kv,
                                       page_size=slot.page_size, write_kv=slot.writes_cache,
                                       rot_amplitude=self.rot_amplitude)
-            q = self.up_q(cq)                                                 # [T, H (dim + rot)] float32
-        else:                                                                 # the queries lead the fused product
-            ops.latent_down_post(down[:, self._lead: self._lead + tail], q_rank=0, rank=self.kv_rank, rot=self.rot_dim,
-                                 rot_dims=self.rot_dims, q_norm_weight=None, c_norm_weight=self.c_norm_weight,
-                                 eps=self.eps, positions=ctx.positions, row_req=ctx.row_request, block_table=table,
-                                 inv_freq=self.inv_freq, kv_layer=slot.kv, page_size=slot.page_size,
-                                 write_kv=slot.writes_cache, rot_amplitude=self.rot_amplitude)
-            q = down[:, : self._lead]
+        # [T, H (dim + rot)] float32: from the query latent, or leading the fused product
+        q = self.up_q(cq) if self.q_rank > 0 else down[:, : self._lead]
         q_plain = ops.head_major(q, heads=H, stride=self.dim + self.rot_dim, col0=0, n=self.dim, out_dtype=act)
         qa = self.up_k.per_group(q_plain, T)                                  # [H T, kv_rank] float32
         qj = ops.latent_q_join(qa, q, ctx.positions, self.inv_freq, heads=H, dim=self.dim, rank=self.kv_rank,

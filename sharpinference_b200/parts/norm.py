@@ -5,15 +5,32 @@ RMSNorm: ``x * rsqrt(mean(x^2) + eps) * w`` (src/SharpInference.Cpu/SimdKernels.
 the weightless form drops ``w`` (src/SharpInference.Cpu/SimdKernels.cs:4252-4283).  The sum of
 squares, the rsqrt and the scaling are float32.  Models that store the weight around zero and scale by
 ``1 + w`` pass ``unit_offset=True``: the sum is formed once, in float32, when the part is built.
+
+A sublayer's output may itself be normed before it enters the stream.  Such an update travels as a :class:`NormedUpdate`
+and the RMS norm that reads the stream next forms both in one kernel.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
 
 from ..kernels import ops
 from .base import Norm, register_part
+
+
+@dataclass
+class NormedUpdate:
+    """``y / sqrt(mean(y^2) + eps) * weight``, an update of the residual stream that is not yet added to it."""
+
+    y: torch.Tensor
+    weight: torch.Tensor
+    eps: float
+
+    def value(self) -> torch.Tensor:
+        """The update itself (tracing only; plain tensor code)."""
+        return self.y * torch.rsqrt(self.y.square().mean(dim=-1, keepdim=True) + self.eps) * self.weight
 
 
 @register_part("norm", "rmsnorm")
@@ -24,6 +41,10 @@ class RMSNorm(Norm):
         self.unit_offset = bool(unit_offset)
 
     def apply(self, x, delta, *, rows=None, out_dtype=torch.bfloat16, want_fp32=False):
+        if isinstance(delta, NormedUpdate):
+            if delta.eps != self.eps:
+                raise ValueError(f"the update's eps ({delta.eps}) and the norm's ({self.eps}) differ")
+            return ops.add_normed(x, delta.y, delta.weight, self.weight, self.eps, out_dtype, rows=rows, want_fp32=want_fp32)
         return ops.add_rmsnorm(x, delta, self.weight, self.eps, out_dtype, rows=rows, want_fp32=want_fp32)
 
 
