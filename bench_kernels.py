@@ -19,6 +19,9 @@
     python bench_kernels.py lightning --batch 64 --tokens 1        (linear attention and its gated norm; --batch 1 --tokens 2048)
     python bench_kernels.py qkv_conv --tokens 2048                 (convolution, rotation, cache write)
     python bench_kernels.py softmax_mixture --tokens 2048          (router with groups, combine with identity experts)
+    python bench_kernels.py delta --batch 64 --tokens 1            (delta rule and its gated norm; --batch 1 --tokens 2048)
+    python bench_kernels.py delta_prep --tokens 2048               (convolution, unit norms, steps, low-rank columns)
+    python bench_kernels.py sandwich --tokens 2048                 (normed update and norm, side gate, element gate, router)
     python bench_kernels.py elementwise --op add_rmsnorm_pair --tokens 2048 --hidden 2048
     python bench_kernels.py elementwise --op add_layernorm --tokens 2048 --hidden 2048
 
@@ -524,6 +527,103 @@ def lightning(ns) -> None:
           f"{2 * B * per_request * 4 / ms / 1e6:.0f} GB/s (read and written once), {4.0 * T * per_request / ms / 1e9:.2f} TFLOP/s float32")
 
 
+def delta(ns) -> None:
+    """The gated delta rule with a decay per key channel and the norm and gate behind it for `batch` requests of `tokens` rows
+    each: per row and head 7 d dv flops (decay, S^T k, update, S^T q: what the recurrence asks for, whatever form runs it);
+    decode streams the state once."""
+    from sharpinference_b200.parts.delta import DeltaPlanner
+    B, n, heads, d, dv = ns.batch, ns.tokens, ns.heads, ns.key_dim, ns.value_dim
+    G = ns.kv_heads or heads
+    T, C = B * n, 2 * G * d + heads * dv
+    qkv = torch.randn(T, C, device=DEV)
+    qk = qkv[:, : 2 * G * d].view(T, 2 * G, d)
+    qk /= qk.norm(dim=-1, keepdim=True)
+    beta = torch.rand(T, heads, device=DEV)
+    z = torch.randn(T, heads * (d + dv), device=DEV)
+    dt_bias, a_log, w = torch.randn(heads * d, device=DEV) - 3, torch.zeros(heads, device=DEV), torch.ones(dv, device=DEV)
+    per_request = ops.delta_state_floats(heads, d, dv)
+    copies = max(1, (300 << 20) // (B * per_request * 4) + 1) if n == 1 else 1
+    state = torch.zeros(copies * B, per_request, device=DEV)
+    offs = torch.arange(0, T + 1, n, dtype=torch.int32, device=DEV)
+    slot_sets = [torch.arange(c * B, (c + 1) * B, dtype=torch.int32, device=DEV) for c in range(copies)]
+    planner = DeltaPlanner(4, True)
+    if ns.walk:
+        planner.WALK_ROWS_UP_TO = 1 << 30
+    if ns.chunk:
+        planner.WALK_ROWS_UP_TO = 0
+    plan = planner.plan([0] * B, [n] * B)
+    dev = {k: (torch.from_numpy(v).to(DEV) if v.size else None) for k, v in plan.arrays.items()}
+    it = {"i": 0}
+
+    def fn():
+        slots = slot_sets[it["i"] % copies]
+        it["i"] += 1
+        y = ops.delta_rule(qkv, beta, z[:, : heads * d], dt_bias=dt_bias, a_log=a_log, row_offsets=offs, state_slots=slots, state=state,
+                           kv_heads=G, heads=heads, d=d, dv=dv, num_requests=B, walk_requests=dev["walk"],
+                           num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"], max_rows=n)
+        ops.head_norm_gate(y, z[:, heads * d:], w, 1e-6, heads, torch.bfloat16)
+    ms = _time(fn, max(ns.iters, copies))
+    print(f"delta batch={B} tokens={n} heads={heads}/{G} d={d} dv={dv}{' walked' if ns.walk else ''}: {ms * 1e3:.1f} us, state "
+          f"{2 * B * per_request * 4 / ms / 1e6:.0f} GB/s (read and written once), {7.0 * T * heads * d * dv / ms / 1e9:.2f} TFLOP/s float32")
+
+
+def delta_prep(ns) -> None:
+    """Convolution, silu, unit norms, steps and low-rank columns behind the delta rule's fused projection."""
+    from sharpinference_b200.parts.delta import DeltaPlanner, delta_columns
+    B, n, heads, d, dv, low = ns.batch, ns.tokens, ns.heads, ns.key_dim, ns.value_dim, 2 * ns.key_dim
+    G = ns.kv_heads or heads
+    C, _, width = delta_columns(G, heads, d, dv, low)
+    T = B * n
+    copies = max(2, (300 << 20) // (T * width * 4) + 1) if T > 64 else 2
+    projs = [torch.randn(T, width, device=DEV) for _ in range(copies)]
+    conv, state = torch.randn(4, C, device=DEV), torch.zeros(B, 3 * C, device=DEV)
+    offs = torch.arange(0, T + 1, n, dtype=torch.int32, device=DEV)
+    slots = torch.arange(B, dtype=torch.int32, device=DEV)
+    arr = DeltaPlanner(4, True).plan([0] * B, [n] * B).arrays["tiles"]
+    tiles = torch.from_numpy(arr).to(DEV) if arr.size else None
+    it = {"i": 0}
+
+    def fn():
+        ops.delta_prep(projs[it["i"] % copies], conv_weight=conv, conv_state=state, row_offsets=offs, state_slots=slots, tiles=tiles,
+                       kv_heads=G, heads=heads, d=d, dv=dv, low=low, act_dtype=torch.bfloat16)
+        it["i"] += 1
+    ms = _time(fn, max(ns.iters, copies))
+    print(f"delta_prep batch={B} tokens={n} heads={heads}/{G} d={d} dv={dv}: {ms * 1e3:.1f} us, "
+          f"{T * (C * 8 + low * 6 + heads * 8) / ms / 1e6:.0f} GB/s")
+
+
+def sandwich(ns) -> None:
+    """A normed update and the norm behind it, the same with the bare stream, the side gate, the element gate of latent
+    attention and the router with sigmoid scores in groups."""
+    T, H, N, k = ns.tokens, ns.hidden, ns.experts, ns.top
+    copies = max(2, (300 << 20) // (T * H * 8) + 1)
+    xs = [(torch.randn(T, H, device=DEV), torch.randn(T, H, device=DEV)) for _ in range(copies)]
+    w1, w2 = torch.ones(H, device=DEV), torch.ones(H, device=DEV)
+    it = {"i": 0}
+
+    def timed(name, fn, nbytes):
+        def call():
+            fn(it["i"] % copies)
+            it["i"] += 1
+        ms = _time(call, max(ns.iters, copies))
+        print(f"{name} tokens={T} hidden={H}: {ms * 1e3:.1f} us, {nbytes / ms / 1e6:.0f} GB/s")
+    timed("add_normed", lambda i: ops.add_normed(xs[i][0], xs[i][1], w1, w2, 1e-6, torch.bfloat16), T * H * 14)
+    timed("add_normed, bare stream", lambda i: ops.add_normed(xs[i][0], xs[i][1], w1, None, 1e-6, torch.bfloat16), T * H * 14)
+    timed("add_rmsnorm", lambda i: ops.add_rmsnorm(xs[i][0], xs[i][1], w1, 1e-6, torch.bfloat16), T * H * 14)
+    n = max(8, H // 16)
+    gate, table = torch.randn(T, n, device=DEV), torch.randn(32768, 10 * n, device=DEV).to(torch.bfloat16)
+    ids = torch.randint(0, 32768, (T,), device=DEV, dtype=torch.int32)
+    timed(f"side_gate n={n}", lambda i: ops.side_gate(gate, ids, table, 3 * n, n, torch.bfloat16), T * n * 8)
+    heads = max(1, H // 128)
+    v, wide = torch.randn(heads * T, 128, device=DEV), torch.randn(T, 2 * H, device=DEV)
+    timed("head_minor, element gate", lambda i: ops.head_minor(v, heads=heads, out_dtype=torch.bfloat16, gate=wide[:, H:]), T * H * 10)
+    timed("head_minor, head gate", lambda i: ops.head_minor(v, heads=heads, out_dtype=torch.bfloat16, gate=wide[:, :heads]), T * H * 6)
+    wr, corr = torch.randn(N, H, device=DEV) * 0.05, torch.randn(N, device=DEV) * 0.1
+    timed(f"router_groups, sigmoid, {N} experts", lambda i: ops.router_groups(
+        xs[i][0], wr, k, correction=corr, renormalize=False, n_groups=4, keep=2, scoring="sigmoid", group_top=2), T * H * 4 + N * H * 4)
+    timed(f"router_topk, {N} experts", lambda i: ops.router_topk(xs[i][0], wr, k, correction=corr), T * H * 4 + N * H * 4)
+
+
 def qkv_conv(ns) -> None:
     """Short convolution of q, k and v, rotation, q store and cache write for `batch` requests of `tokens` rows each."""
     from sharpinference_b200.parts.position import leading_rotary_inv_freq_parts
@@ -768,6 +868,23 @@ def main(argv=None) -> int:
     p.add_argument("--value-dim", type=int, default=128)
     p.add_argument("--walk", action="store_true", help="walk the rows one by one whatever their number")
     p.set_defaults(fn=lightning)
+    for name, fn in (("delta", delta), ("delta_prep", delta_prep)):
+        p = sub.add_parser(name)
+        p.add_argument("--batch", type=int, default=64 if name == "delta" else 1)
+        p.add_argument("--tokens", type=int, default=1 if name == "delta" else 2048)
+        p.add_argument("--heads", type=int, default=16)
+        p.add_argument("--kv-heads", type=int, default=0, help="heads of q and k (0: as many as heads)")
+        p.add_argument("--key-dim", type=int, default=128)
+        p.add_argument("--value-dim", type=int, default=128)
+        p.add_argument("--walk", action="store_true", help="walk the rows one by one whatever their number")
+        p.add_argument("--chunk", action="store_true", help="cut into chunks whatever the number of rows")
+        p.set_defaults(fn=fn)
+    p = sub.add_parser("sandwich")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--hidden", type=int, default=2048)
+    p.add_argument("--experts", type=int, default=16)
+    p.add_argument("--top", type=int, default=2)
+    p.set_defaults(fn=sandwich)
     p = sub.add_parser("qkv_conv")
     p.add_argument("--batch", type=int, default=1)
     p.add_argument("--tokens", type=int, default=2048)

@@ -235,7 +235,9 @@ constexpr int WALK_LANES = 8;                                  // lanes of a col
 constexpr int WALK_COLS = WALK_THREADS / WALK_LANES;
 constexpr int WALK_STAGE = 8;                                  // rows staged together (one warp each forms k . q)
 
-template <int R4>                                              // float4 of a column a lane: 32 R4 >= d
+// A walk over many rows (LONG) starts on an empty GPU and lets nothing onto its SMs: its few blocks would otherwise land
+// several to an SM.
+template <int R4, bool LONG>                                   // float4 of a column a lane: 32 R4 >= d
 __global__ void __launch_bounds__(WALK_THREADS) delta_walk_kernel(DeltaArgs a) {
     constexpr int DP = 32 * R4;
     extern __shared__ __align__(16) float walk_smem[];
@@ -247,7 +249,8 @@ __global__ void __launch_bounds__(WALK_THREADS) delta_walk_kernel(DeltaArgs a) {
     float* b_s = o_s + WALK_STAGE * WALK_COLS;                 // [STAGE] beta, [STAGE] k . q
     const int h = blockIdx.y, hk = h / (a.heads / a.kvh);
     const float rate = expf(a.a_log[h]);
-    pdl_wait();
+    if (LONG) pdl_wait_only();
+    else pdl_wait();
     const int req = a.requests ? a.requests[blockIdx.z] : blockIdx.z;
     const int first = a.row_offsets[req], rows = a.row_offsets[req + 1] - first;
     if (rows <= 0) return;
@@ -345,35 +348,42 @@ static bool fill_delta(DeltaArgs& a, const float* qkv, const float* beta, const 
 }
 
 template <int R4>
-static int launch_delta_walk(const DeltaArgs& a, int n, cudaStream_t stream) {
+static int launch_delta_walk(const DeltaArgs& a, int n, int max_rows, cudaStream_t stream) {
     const dim3 grid((a.dv + WALK_COLS - 1) / WALK_COLS, a.heads, n);
     const size_t smem = (size_t)(WALK_STAGE * (3 * 32 * R4 + 2 * WALK_COLS) + 2 * WALK_STAGE) * sizeof(float);
     static bool configured = false;
     if (smem > 48 * 1024 && !configured) {
-        if (cudaFuncSetAttribute(delta_walk_kernel<R4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(delta_walk_kernel<R4, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(delta_walk_kernel<R4, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return SHARPI_LAUNCH_FAILED;
         configured = true;
     }
-    SHARPI_LAUNCH_PDL(delta_walk_kernel<R4>, grid, WALK_THREADS, smem, stream, a);
+    if (max_rows > WALK_STAGE) {
+        delta_walk_kernel<R4, true><<<grid, WALK_THREADS, smem, stream>>>(a);
+        SHARPI_CHECK_LAUNCH();
+    } else {
+        SHARPI_LAUNCH_PDL((delta_walk_kernel<R4, false>), grid, WALK_THREADS, smem, stream, a);
+    }
     return SHARPI_OK;
 }
 
-// `requests` (nullable): the `n` requests of the step to serve; null: requests 0 .. n - 1.
+// `requests` (nullable): the `n` requests of the step to serve; null: requests 0 .. n - 1.  `max_rows`: the most rows one of
+// them brings (how the kernel is launched; no result depends on it).
 SHARPI_API int sharpi_delta_walk(const float* qkv, const float* beta, const float* z, int ldz, const float* dt_bias,
                                  const float* a_log, const int* row_offsets, const int* state_slots, const int* requests,
-                                 int n, float* state, long long state_stride, float* y, int kvh, int heads, int d, int dv,
-                                 cudaStream_t stream) {
+                                 int n, int max_rows, float* state, long long state_stride, float* y, int kvh, int heads,
+                                 int d, int dv, cudaStream_t stream) {
     if (n <= 0) return SHARPI_OK;
     DeltaArgs a;
     if (n > 65535 || !fill_delta(a, qkv, beta, z, ldz, dt_bias, a_log, row_offsets, state_slots, state, state_stride, y, kvh,
                                  heads, d, dv))
         return SHARPI_BAD_ARGUMENT;
     a.requests = requests;
-    if (d <= 32) return launch_delta_walk<1>(a, n, stream);
-    if (d <= 64) return launch_delta_walk<2>(a, n, stream);
-    if (d <= 128) return launch_delta_walk<4>(a, n, stream);
-    if (d <= 256) return launch_delta_walk<8>(a, n, stream);
-    return launch_delta_walk<16>(a, n, stream);
+    if (d <= 32) return launch_delta_walk<1>(a, n, max_rows, stream);
+    if (d <= 64) return launch_delta_walk<2>(a, n, max_rows, stream);
+    if (d <= 128) return launch_delta_walk<4>(a, n, max_rows, stream);
+    if (d <= 256) return launch_delta_walk<8>(a, n, max_rows, stream);
+    return launch_delta_walk<16>(a, n, max_rows, stream);
 }
 
 // -------------------------------------------------------------------------------------------------------------
@@ -398,7 +408,7 @@ __device__ __forceinline__ float transpose_sum32(float (&acc)[32], int lane) {
 }
 
 // (1) one chunk of one head
-__global__ void __launch_bounds__(DC_THREADS) delta_chunk_kernel(DeltaArgs a) {
+__global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_kernel(DeltaArgs a) {
     extern __shared__ __align__(16) float chunk_smem[];
     const int ldk = a.d;
     float* k_s = chunk_smem;                                   // [DC_ROWS][d] each
@@ -705,7 +715,9 @@ SHARPI_API int sharpi_delta_chunks(const float* qkv, const float* beta, const fl
         configured = true;
     }
     SHARPI_LAUNCH_PDL(delta_chunk_kernel, dim3(n_chunks, heads), DC_THREADS, smem1, stream, a);
-    SHARPI_LAUNCH_PDL(delta_carry_kernel, dim3((dv + DC_COLS - 1) / DC_COLS, heads, n_spans), DC_THREADS, smem2, stream, a);
+    // the plain way: its blocks run long and are to lie evenly over an empty GPU
+    delta_carry_kernel<<<dim3((dv + DC_COLS - 1) / DC_COLS, heads, n_spans), DC_THREADS, smem2, stream>>>(a);
+    SHARPI_CHECK_LAUNCH();
     return SHARPI_OK;
 }
 

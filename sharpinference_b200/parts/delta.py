@@ -56,7 +56,7 @@ class DeltaPlanner(StepPlanner):
                 spans.append((b, len(chunks), (n + ops.DELTA_CHUNK - 1) // ops.DELTA_CHUNK, 0))
                 chunks.extend((first + r, min(ops.DELTA_CHUNK, n - r), b, 0) for r in range(0, n, ops.DELTA_CHUNK))
             first += n
-        num_walk = len(walk)
+        num_walk, walk_rows = len(walk), max((lengths[b] for b in walk), default=0)
         if not spans:
             walk = []
         if len(tiles) == len(lengths):
@@ -65,7 +65,7 @@ class DeltaPlanner(StepPlanner):
                                     "walk": np.asarray(walk, dtype=np.int32),
                                     "chunks": np.asarray(chunks, dtype=np.int32).reshape(-1, 4),
                                     "spans": np.asarray(spans, dtype=np.int32).reshape(-1, 4)},
-                            values={"num_walk": num_walk})
+                            values={"num_walk": num_walk, "walk_rows": walk_rows})
 
 
 @register_part("mixer", "channel_delta")
@@ -116,5 +116,6 @@ class ChannelDelta(Mixer):
         n = self.heads * self.dim
         y = ops.delta_rule(qkv, beta, z[:, :n], dt_bias=self.dt_bias, a_log=self.a_log, row_offsets=ctx.row_offsets,
                            state_slots=ctx.state_slots, state=slot.states["S"], num_requests=ctx.num_requests,
-                           walk_requests=plan.walk, num_walk=plan.num_walk, chunks=plan.chunks, spans=plan.spans, **sizes)
+                           walk_requests=plan.walk, num_walk=plan.num_walk, chunks=plan.chunks, spans=plan.spans,
+                           max_rows=plan.walk_rows, **sizes)
         return self.out(ops.head_norm_gate(y, z[:, n:], self.norm_weight, self.eps, self.heads, self.act_dtype))
