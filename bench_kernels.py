@@ -560,7 +560,7 @@ def delta(ns) -> None:
         it["i"] += 1
         y = ops.delta_rule(qkv, beta, z[:, : heads * d], dt_bias=dt_bias, a_log=a_log, row_offsets=offs, state_slots=slots, state=state,
                            kv_heads=G, heads=heads, d=d, dv=dv, num_requests=B, walk_requests=dev["walk"],
-                           num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"], max_rows=n)
+                           num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"], max_rows=n, split=not ns.exact)
         ops.head_norm_gate(y, z[:, heads * d:], w, 1e-6, heads, torch.bfloat16)
     ms = _time(fn, max(ns.iters, copies))
     print(f"delta batch={B} tokens={n} heads={heads}/{G} d={d} dv={dv}{' walked' if ns.walk else ''}: {ms * 1e3:.1f} us, state "
@@ -877,6 +877,7 @@ def main(argv=None) -> int:
         p.add_argument("--key-dim", type=int, default=128)
         p.add_argument("--value-dim", type=int, default=128)
         p.add_argument("--walk", action="store_true", help="walk the rows one by one whatever their number")
+        p.add_argument("--exact", action="store_true", help="chunks in float32 FMAs")
         p.add_argument("--chunk", action="store_true", help="cut into chunks whatever the number of rows")
         p.set_defaults(fn=fn)
     p = sub.add_parser("sandwich")

@@ -24,9 +24,12 @@
 //                        chunks: one product with S_0 for all of a chunk's rows and one back into the state.
 //   sharpi_head_norm_gate  out = y / sqrt(mean over the head (y^2) + eps) * w * sigmoid(gate)
 //
-// Everything is float32 FMAs.  A request's form (walk or chunks) and its chunks depend on its own rows alone, and no sum
+// Everything is float32.  The chunks' walk is float32 FMAs, or (`split`, key sizes that are multiples of 64) tensor-core
+// products of operands cut into three bfloat16 pieces each, 24 bits in all, of which the six products above 2^-24 are
+// formed and added in float32; the state itself stays float32 in registers.  A request's form (walk or chunks) and its chunks depend on its own rows alone, and no sum
 // depends on what else is in the step.  State per request and head: dv columns of dp = d rounded up to 4 floats.
 #include "common.cuh"
+#include "mma_sync.cuh"
 
 constexpr int DELTA_MAX_KEY = 512;        // walk
 constexpr int DELTA_MAX_CHUNK_KEY = 256;  // chunks
@@ -224,7 +227,8 @@ struct DeltaArgs {
     float* state;               // [slots][heads][dv][dp]
     long long state_stride;
     float* y;                   // [T, heads * dv]
-    float* mats;                // chunks: [n][heads][dp][48]: -W | D q - B W | decayed keys, a key channel's rows together
+    float* mats;                // chunks: [n][heads][dp][48]: -W | D q - B W | decayed keys, a key channel's rows together;
+                                // split: [n][heads][73 dp] words, the operands of the tensor-core walk (delta_carry_mma)
     float* last;                // chunks: [n][heads][dp]: the product of all decays of the chunk
     float* u0;                  // chunks: [n][heads][DC_ROWS][dv]
     int kvh, heads, d, dp, dv, C;
@@ -407,139 +411,188 @@ __device__ __forceinline__ float transpose_sum32(float (&acc)[32], int lane) {
     return acc[0];
 }
 
+// Two neighbouring elements in three bfloat16 pieces each (24 bits together), packed as an operand register.
+struct Pieces {
+    uint32_t v[3];
+};
+__device__ __forceinline__ Pieces split3(float x, float y) {
+    Pieces r;
+#pragma unroll
+    for (int p = 0; p < 3; ++p) {
+        r.v[p] = mma16::pack_bf16(x, y);
+        if (p < 2) {
+            x -= __uint_as_float(r.v[p] << 16);
+            y -= __uint_as_float(r.v[p] & 0xffff0000u);
+        }
+    }
+    return r;
+}
+
+// The operands of the tensor-core walk in the order in which its lanes (g = lane / 4, t = lane % 4) take them, 16 bytes each.
+// Of the 32 rows -W | D q - B W, per 16 key channels, piece and pair of row tiles: words (tile 0: channels 2t, 2t + 1 of
+// row g | the same 8 further | tile 1 likewise); of the decayed keys, per 16 key channels and piece: (channel g: rows 2t,
+// 2t + 1 | 8 further | channel g + 8 likewise); then the dp products of decays.
+constexpr int CM_M_WORDS = 3 * 2 * 128, CM_K_WORDS = 3 * 128;  // of 16 key channels
+__host__ __device__ constexpr int cm_words(int dp) { return dp / 16 * (CM_M_WORDS + CM_K_WORDS) + dp; }
+__device__ __forceinline__ int cm_m_half(int p, int row, int key) {            // index of a bfloat16
+    const int k = key & 15, n = row >> 3;
+    const int word = ((key >> 4) * 6 + p * 2 + (n >> 1)) * 128 + ((row & 7) * 4 + ((k & 7) >> 1)) * 4 + (n & 1) * 2 + (k >> 3);
+    return 2 * word + (k & 1);
+}
+__device__ __forceinline__ int cm_k_word(int dp, int p, int pair, int key) {   // rows 2 pair, 2 pair + 1
+    return dp / 16 * CM_M_WORDS + ((key >> 4) * 3 + p) * 128 + ((key & 7) * 4 + (pair & 3)) * 4 + ((key >> 3) & 1) * 2 + (pair >> 2);
+}
+
 // (1) one chunk of one head
-__global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_kernel(DeltaArgs a) {
+template <bool SPLIT>
+__global__ void __launch_bounds__(DC_THREADS, SPLIT ? 3 : 2) delta_chunk_kernel(DeltaArgs a) {
     extern __shared__ __align__(16) float chunk_smem[];
-    const int ldk = a.d;
-    float* k_s = chunk_smem;                                   // [DC_ROWS][d] each
-    float* q_s = k_s + DC_ROWS * ldk;
-    float* g_s = q_s + DC_ROWS * ldk;
-    __shared__ __align__(16) float A_s[DC_ROWS][DC_ROWS];      // [t][s]: beta_t A_ts, zeros from the diagonal on
-    __shared__ __align__(16) float B_s[DC_ROWS][DC_ROWS];      // [t][s], zeros above the diagonal
+    const int d = a.d, dp = a.dp;
+    float* k_s = chunk_smem;                                   // [DC_ROWS][dp] each
+    float* q_s = k_s + DC_ROWS * dp;
+    float* g_s = q_s + DC_ROWS * dp;
+    uint32_t* ops_s = reinterpret_cast<uint32_t*>(g_s + DC_ROWS * dp);         // SPLIT: cm_words(dp)
+    __shared__ __align__(16) float A_s[DC_ROWS][DC_ROWS];      // [s][t]: beta_t A_ts where t > s
+    __shared__ __align__(16) float B_s[DC_ROWS][DC_ROWS];      // [s][t]: B_ts where t >= s
     __shared__ float b_s[DC_ROWS];
     const int h = blockIdx.y, hk = h / (a.heads / a.kvh);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float rate = expf(a.a_log[h]);
     pdl_wait();
     const int chunk = blockIdx.x;
     const int row0 = a.chunks[4 * chunk], rows = a.chunks[4 * chunk + 1];
-    const int d = a.d;
-    for (int i = threadIdx.x; i < DC_ROWS * d; i += DC_THREADS) {
-        const int r = i / d, e = i % d;
-        float q = 0.0f, k = 0.0f, g = 1.0f;                    // rows behind the chunk's last leave everything as it is
-        if (r < rows) {
-            const size_t t = row0 + r;
-            const float* row = a.qkv + t * a.C;
-            q = row[hk * d + e];
-            k = row[(a.kvh + hk) * d + e];
-            g = delta_decay(a.z[t * a.ldz + h * d + e] + a.dt_bias[h * d + e], rate);
+#pragma unroll
+    for (int r = warp; r < DC_ROWS; r += DC_THREADS / 32) {
+        const size_t t = row0 + min(r, rows - 1);
+        const float* row = a.qkv + t * a.C + hk * d;
+        const float* z = a.z + t * a.ldz + h * d;
+        const bool live = r < rows;                            // rows behind the chunk's last leave everything as it is
+#pragma unroll 4
+        for (int e = lane; e < dp; e += 32) {
+            const bool in = e < d;
+            const float q = in ? row[e] : 0.0f, k = in ? row[a.kvh * d + e] : 0.0f;
+            const float g = in ? z[e] + a.dt_bias[h * d + e] : 0.0f;
+            q_s[r * dp + e] = live ? q : 0.0f;
+            k_s[r * dp + e] = live ? k : 0.0f;
+            g_s[r * dp + e] = live ? delta_decay(g, rate) : 1.0f;
         }
-        q_s[i] = q; k_s[i] = k; g_s[i] = g;
     }
     if (threadIdx.x < DC_ROWS)
         b_s[threadIdx.x] = threadIdx.x < rows ? a.beta[(size_t)(row0 + threadIdx.x) * a.heads + h] : 0.0f;
     __syncthreads();
-    {   // A and B: warp w forms the columns s = 2w, 2w + 1; a lane walks its channels down the rows
-        const int s0 = 2 * (threadIdx.x >> 5), lane = threadIdx.x & 31;
-        float acc0[32], acc1[32];                              // [t] A, [16 + t] B
+    // A and B: warp w forms the columns s = w and 15 - w (17 rows in all); a lane walks its channels down the rows
+#pragma unroll 1
+    for (int s = warp; s < DC_ROWS; s += DC_ROWS - 1 - 2 * warp) {
+        float acc[32];                                         // [t] A, [16 + t] B
 #pragma unroll
-        for (int i = 0; i < 32; ++i) acc0[i] = acc1[i] = 0.0f;
-        for (int e = lane; e < d; e += 32) {
-            float p0 = k_s[s0 * d + e], p1 = 0.0f;
+        for (int i = 0; i < 32; ++i) acc[i] = 0.0f;
+        for (int e = lane; e < dp; e += 32) {
+            float p = k_s[s * dp + e];
 #pragma unroll
             for (int t = 0; t < DC_ROWS; ++t) {
-                if (t < s0) continue;
-                const float k = k_s[t * d + e], q = q_s[t * d + e], g = g_s[t * d + e];
-                if (t > s0) p0 *= g;
-                if (t == s0 + 1) p1 = k;
-                if (t > s0 + 1) p1 *= g;
-                acc0[t] = fmaf(k, p0, acc0[t]);
-                acc0[16 + t] = fmaf(q, p0, acc0[16 + t]);
-                acc1[t] = fmaf(k, p1, acc1[t]);
-                acc1[16 + t] = fmaf(q, p1, acc1[16 + t]);
+                if (t < s) continue;
+                if (t > s) p *= g_s[t * dp + e];
+                acc[t] = fmaf(k_s[t * dp + e], p, acc[t]);
+                acc[16 + t] = fmaf(q_s[t * dp + e], p, acc[16 + t]);
             }
         }
-        const float m0 = transpose_sum32(acc0, lane), m1 = transpose_sum32(acc1, lane);
-        const int t = lane & 15;
-        if (lane < 16) {
-            A_s[t][s0] = t > s0 ? b_s[t] * m0 : 0.0f;
-            A_s[t][s0 + 1] = t > s0 + 1 ? b_s[t] * m1 : 0.0f;
-        } else {
-            B_s[t][s0] = t >= s0 ? m0 : 0.0f;
-            B_s[t][s0 + 1] = t >= s0 + 1 ? m1 : 0.0f;
-        }
+        const float m = transpose_sum32(acc, lane);
+        if (lane < 16) A_s[s][lane] = b_s[lane] * m;
+        else B_s[s][lane - 16] = m;
+        if (s == DC_ROWS - 1 - warp) break;
     }
     __syncthreads();
-    // a thread a column of [D k | v]: solve, then multiply by B
+    // a thread a column of [D k | v]: w <- the triangular system's solution, row by row into all rows below it, and b += B w
     const size_t at = (size_t)chunk * a.heads + h;
-    for (int j = threadIdx.x; j < a.dp + a.dv; j += DC_THREADS) {
+    for (int j = threadIdx.x; j < dp + a.dv; j += DC_THREADS) {
         float w[DC_ROWS], b[DC_ROWS];
-        if (j < a.dp) {
+        const bool key = j < dp;
+        if (key) {
             float D = 1.0f;
 #pragma unroll
             for (int t = 0; t < DC_ROWS; ++t) {
-                if (j < d) D *= g_s[t * d + j];
-                w[t] = j < d ? D * k_s[t * d + j] : 0.0f;
-                b[t] = j < d ? D * q_s[t * d + j] : 0.0f;
+                D *= g_s[t * dp + j];
+                w[t] = -b_s[t] * (D * k_s[t * dp + j]);        // the key columns are kept negated: -W
+                b[t] = D * q_s[t * dp + j];
             }
-            a.last[at * a.dp + j] = D;
+            if (SPLIT) ops_s[cm_words(dp) - dp + j] = __float_as_uint(D);
+            else a.last[at * dp + j] = D;
         } else {
+            const float* v = a.qkv + (size_t)row0 * a.C + 2 * a.kvh * d + (size_t)h * a.dv + j - dp;
 #pragma unroll
             for (int t = 0; t < DC_ROWS; ++t) {
-                w[t] = t < rows ? a.qkv[(size_t)(row0 + t) * a.C + 2 * a.kvh * d + (size_t)h * a.dv + j - a.dp] : 0.0f;
+                w[t] = t < rows ? b_s[t] * v[(size_t)t * a.C] : 0.0f;
                 b[t] = 0.0f;
             }
         }
 #pragma unroll
-        for (int t = 0; t < DC_ROWS; ++t) {
-            float acc = b_s[t] * w[t];
+        for (int r = 0; r < DC_ROWS; ++r) {
 #pragma unroll
-            for (int s4 = 0; s4 < t; s4 += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(&A_s[t][s4]);
-                if (s4 < t) acc = fmaf(-m.x, w[s4], acc);
-                if (s4 + 1 < t) acc = fmaf(-m.y, w[s4 + 1], acc);
-                if (s4 + 2 < t) acc = fmaf(-m.z, w[s4 + 2], acc);
-                if (s4 + 3 < t) acc = fmaf(-m.w, w[s4 + 3], acc);
+            for (int t4 = r / 4 * 4; t4 < DC_ROWS; t4 += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(&A_s[r][t4]);
+                const float4 n = *reinterpret_cast<const float4*>(&B_s[r][t4]);
+                if (t4 > r) w[t4] = fmaf(-m.x, w[r], w[t4]);
+                if (t4 + 1 > r) w[t4 + 1] = fmaf(-m.y, w[r], w[t4 + 1]);
+                if (t4 + 2 > r) w[t4 + 2] = fmaf(-m.z, w[r], w[t4 + 2]);
+                if (t4 + 3 > r) w[t4 + 3] = fmaf(-m.w, w[r], w[t4 + 3]);
+                if (t4 >= r) b[t4] = fmaf(n.x, w[r], b[t4]);
+                if (t4 + 1 >= r) b[t4 + 1] = fmaf(n.y, w[r], b[t4 + 1]);
+                if (t4 + 2 >= r) b[t4 + 2] = fmaf(n.z, w[r], b[t4 + 2]);
+                if (t4 + 3 >= r) b[t4 + 3] = fmaf(n.w, w[r], b[t4 + 3]);
             }
-            w[t] = acc;
         }
-        const float sign = j < a.dp ? -1.0f : 1.0f;
+        if (!key) {
+            float* u0 = a.u0 + at * DC_ROWS * a.dv + j - dp;
+            float* y = a.y + ((size_t)row0 * a.heads + h) * a.dv + j - dp;
 #pragma unroll
-        for (int t = 0; t < DC_ROWS; ++t) {
-            float acc = 0.0f;
-#pragma unroll
-            for (int s4 = 0; s4 <= t; s4 += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(&B_s[t][s4]);
-                acc = fmaf(m.x, w[s4], acc);
-                if (s4 + 1 <= t) acc = fmaf(m.y, w[s4 + 1], acc);
-                if (s4 + 2 <= t) acc = fmaf(m.z, w[s4 + 2], acc);
-                if (s4 + 3 <= t) acc = fmaf(m.w, w[s4 + 3], acc);
+            for (int t = 0; t < DC_ROWS; ++t) {
+                u0[t * a.dv] = w[t];
+                if (t < rows) y[(size_t)t * a.heads * a.dv] = b[t];
             }
-            b[t] = fmaf(sign, acc, b[t]);
+            continue;
         }
-        if (j < a.dp) {
-            float* out = a.mats + (at * a.dp + j) * DC_MATS;
+        float* out = a.mats + (at * dp + j) * DC_MATS;
+        uint16_t* half = reinterpret_cast<uint16_t*>(ops_s);
+        if (SPLIT) {
+#pragma unroll
+            for (int t = 0; t < DC_ROWS; ++t) {                // the two rows of a pair go to different tiles
+                const Pieces x = split3(w[t], b[t]);
+#pragma unroll
+                for (int p = 0; p < 3; ++p) {
+                    half[cm_m_half(p, t, j)] = (uint16_t)x.v[p];
+                    half[cm_m_half(p, DC_ROWS + t, j)] = (uint16_t)(x.v[p] >> 16);
+                }
+            }
+        } else {
 #pragma unroll
             for (int t = 0; t < DC_ROWS; t += 4) {
-                *reinterpret_cast<float4*>(out + t) = make_float4(-w[t], -w[t + 1], -w[t + 2], -w[t + 3]);
+                *reinterpret_cast<float4*>(out + t) = make_float4(w[t], w[t + 1], w[t + 2], w[t + 3]);
                 *reinterpret_cast<float4*>(out + DC_ROWS + t) = make_float4(b[t], b[t + 1], b[t + 2], b[t + 3]);
             }
-            float E = 1.0f;
+        }
+        float E = 1.0f;
 #pragma unroll
-            for (int t = DC_ROWS - 1; t >= 0; --t) {
-                w[t] = j < d ? E * k_s[t * d + j] : 0.0f;
-                if (j < d) E *= g_s[t * d + j];
+        for (int t = DC_ROWS - 1; t >= 0; --t) {
+            w[t] = E * k_s[t * dp + j];
+            E *= g_s[t * dp + j];
+        }
+        if (SPLIT) {
+#pragma unroll
+            for (int t = 0; t < DC_ROWS / 2; ++t) {
+                const Pieces x = split3(w[2 * t], w[2 * t + 1]);
+#pragma unroll
+                for (int p = 0; p < 3; ++p) ops_s[cm_k_word(dp, p, t, j)] = x.v[p];
             }
+        } else {
 #pragma unroll
             for (int t = 0; t < DC_ROWS; t += 4)
                 *reinterpret_cast<float4*>(out + 2 * DC_ROWS + t) = make_float4(w[t], w[t + 1], w[t + 2], w[t + 3]);
-        } else {
-            const int cc = j - a.dp;
-#pragma unroll
-            for (int t = 0; t < DC_ROWS; ++t) {
-                a.u0[(at * DC_ROWS + t) * a.dv + cc] = w[t];
-                if (t < rows) a.y[((size_t)(row0 + t) * a.heads + h) * a.dv + cc] = b[t];
-            }
         }
+    }
+    if (SPLIT) {
+        __syncthreads();
+        uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<uint32_t*>(a.mats) + at * cm_words(dp));
+        for (int i = threadIdx.x; i < cm_words(dp) / 4; i += DC_THREADS) dst[i] = reinterpret_cast<const uint4*>(ops_s)[i];
     }
 }
 
@@ -688,14 +741,221 @@ __global__ void __launch_bounds__(DC_THREADS) delta_carry_kernel(DeltaArgs a) {
     }
 }
 
+// The same on the tensor cores.  A block owns DC_COLS columns of one head's state, a warp 16 KB of the key channels, as S^T
+// in the layout of the accumulators of m16n8k16 (columns of S down, key channels across): two neighbouring tiles are at once
+// the left operand of the product with the chunk's rows, so the state never leaves the registers.
+//   P^T = S^T [-W | D q - B W]^T  (each warp its key channels; the parts are added in shared memory)
+//   S^T <- last * S^T + U^T K     (U^T = U_0^T + P^T's first rows)
+constexpr int CM_PART = 40;               // floats between two columns of a part (8 mod 32: no bank twice)
+
+// acc[n] += a b[n] for N tiles, the six products of the pieces that count, a tile after the other for each of them
+template <int N>
+__device__ __forceinline__ void mma_split(float (*acc)[4], const uint32_t (&x)[3][4], const uint32_t (&b)[3][N][2]) {
+    constexpr int order[6][2] = {{2, 0}, {0, 2}, {1, 1}, {1, 0}, {0, 1}, {0, 0}};
+#pragma unroll
+    for (int o = 0; o < 6; ++o)
+#pragma unroll
+        for (int n = 0; n < N; ++n) mma16::mma_bf16(acc[n], x[order[o][0]], b[order[o][1]][n][0], b[order[o][1]][n][1]);
+}
+
+// Two tiles: the three smaller products in sums of their own, so that no accumulator waits for six products in a row.
+__device__ __forceinline__ void mma_split_pair(float (*acc)[4], const uint32_t (&x)[3][4], const uint32_t (&b)[3][2][2]) {
+    float small[2][4] = {};
+    constexpr int order[3][4] = {{2, 0, 1, 0}, {0, 2, 0, 1}, {1, 1, 0, 0}};
+#pragma unroll
+    for (int o = 0; o < 3; ++o) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n) mma16::mma_bf16(small[n], x[order[o][0]], b[order[o][1]][n][0], b[order[o][1]][n][1]);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) mma16::mma_bf16(acc[n], x[order[o][2]], b[order[o][3]][n][0], b[order[o][3]][n][1]);
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[n][e] += small[n][e];
+}
+
+constexpr int carry_mma_words(int warps, int kb) {             // 32-bit words of shared memory
+    return 2 * cm_words(16 * warps * kb) + warps * DC_COLS * CM_PART + 3 * 128;
+}
+
+template <int WARPS, int KB>
+__global__ void __launch_bounds__(WARPS * 32) delta_carry_mma_kernel(DeltaArgs a) {
+    constexpr int THREADS = WARPS * 32, DP = 16 * WARPS * KB, BUF = cm_words(DP);
+    extern __shared__ __align__(16) uint32_t cm_smem[];
+    float* part_s = reinterpret_cast<float*>(cm_smem + 2 * BUF);               // [WARPS][DC_COLS][CM_PART]
+    uint32_t* u_s = cm_smem + 2 * BUF + WARPS * DC_COLS * CM_PART;             // [3][32 lanes][4]: U^T as a left operand
+    pdl_wait_only();
+    const int* span = a.spans + 4 * blockIdx.z;
+    const int req = span[0], chunk0 = span[1], n_chunks = span[2];
+    const int h = blockIdx.y, c0 = blockIdx.x * DC_COLS, dv = a.dv;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    float* st = a.state + (size_t)a.state_slots[req] * a.state_stride + ((size_t)h * dv + c0) * DP;
+
+    auto fetch = [&](int i) {                                  // chunk i of the span into buffer i & 1
+        const uint32_t* src = reinterpret_cast<const uint32_t*>(a.mats) + ((size_t)(chunk0 + i) * a.heads + h) * BUF + 4 * tid;
+        uint32_t* dst = cm_smem + (i & 1) * BUF + 4 * tid;
+#pragma unroll
+        for (int p = 0; p < (BUF / 4 + THREADS - 1) / THREADS; ++p)
+            if (tid + p * THREADS < BUF / 4) mma16::cp_async_16(dst + 4 * p * THREADS, src + 4 * p * THREADS, 16);
+        mma16::cp_async_commit();
+    };
+    fetch(0);
+    const bool in0 = c0 + g < dv, in1 = c0 + g + 8 < dv;
+    float S[2 * KB][4];
+    float* own = st + (size_t)g * DP + 16 * KB * warp + 2 * t;                 // the warp's key channels
+#pragma unroll
+    for (int n = 0; n < 2 * KB; ++n) {
+        const float2 x = in0 ? *reinterpret_cast<const float2*>(own + 8 * n) : make_float2(0.0f, 0.0f);
+        const float2 y = in1 ? *reinterpret_cast<const float2*>(own + 8 * DP + 8 * n) : make_float2(0.0f, 0.0f);
+        S[n][0] = x.x; S[n][1] = x.y; S[n][2] = y.x; S[n][3] = y.y;
+    }
+    // the closing sums: task (row tile n, column half) of 32 lanes each, a lane rows 8n + 2t, + 1 of column g + 8 half; tiles
+    // 0 and 1 are U, 2 and 3 the outputs
+    constexpr int TASKS = (8 + WARPS - 1) / WARPS;
+    // what the sums start from, asked for a chunk ahead (a portion's chunks lie end to end, all but the last of DC_ROWS rows)
+    const int first = a.chunks[4 * chunk0], total = (n_chunks - 1) * DC_ROWS + a.chunks[4 * (chunk0 + n_chunks - 1) + 1];
+    float* from[TASKS];
+    size_t step[TASKS], next_row[TASKS];                       // to the next chunk, to the second of the two rows
+    float2 base[TASKS], ahead[TASKS];
+#pragma unroll
+    for (int k = 0; k < TASKS; ++k) {
+        const int task = warp + k * WARPS, n = task >> 1, col = c0 + g + 8 * (task & 1), r = 8 * (n & 1) + 2 * t;
+        const bool u = n < 2;
+        next_row[k] = u ? dv : (size_t)a.heads * dv;
+        step[k] = (size_t)DC_ROWS * a.heads * dv;
+        from[k] = u ? a.u0 + (((size_t)chunk0 * a.heads + h) * DC_ROWS + r) * dv + col
+                    : a.y + ((size_t)(first + r) * a.heads + h) * dv + col;
+        if (task >= 8 || col >= dv) from[k] = nullptr;
+    }
+    auto ask = [&](int i) {
+#pragma unroll
+        for (int k = 0; k < TASKS; ++k) {
+            const int n = (warp + k * WARPS) >> 1, r = 8 * (n & 1) + 2 * t;
+            const int left = n < 2 ? DC_ROWS : total - i * DC_ROWS;
+            const float* p = from[k] + i * step[k];
+            ahead[k].x = from[k] && r < left ? p[0] : 0.0f;
+            ahead[k].y = from[k] && r + 1 < left ? p[next_row[k]] : 0.0f;
+        }
+    };
+    ask(0);
+    for (int i = 0; i < n_chunks; ++i) {
+#pragma unroll
+        for (int k = 0; k < TASKS; ++k) base[k] = ahead[k];
+        if (i + 1 < n_chunks) ask(i + 1);
+        mma16::cp_async_wait<0>();
+        __syncthreads();                                       // the chunk is there, and everyone is done with the one before
+        if (i + 1 < n_chunks) fetch(i + 1);
+        const uint4* M = reinterpret_cast<const uint4*>(cm_smem + (i & 1) * BUF) + lane;
+        float P[4][4] = {};                                    // P^T: a tile eight of the 32 rows
+#pragma unroll
+        for (int kb = 0; kb < KB; ++kb) {
+            uint32_t b[3][4][2];
+#pragma unroll
+            for (int p = 0; p < 3; ++p)
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    const uint4 v = M[(((warp * KB + kb) * 3 + p) * 2 + n) * 32];
+                    b[p][2 * n][0] = v.x; b[p][2 * n][1] = v.y; b[p][2 * n + 1][0] = v.z; b[p][2 * n + 1][1] = v.w;
+                }
+            uint32_t x[3][4];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {                      // (g, 2t..), (g + 8, 2t..), (g, 2t + 8..), (g + 8, 2t + 8..)
+                const float* s = S[2 * kb + (r >> 1)] + 2 * (r & 1);
+                const Pieces v = split3(s[0], s[1]);
+                x[0][r] = v.v[0]; x[1][r] = v.v[1]; x[2][r] = v.v[2];
+            }
+            mma_split<4>(P, x, b);
+        }
+        float* part = part_s + warp * DC_COLS * CM_PART + g * CM_PART + 2 * t;
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+            *reinterpret_cast<float2*>(part + 8 * n) = make_float2(P[n][0], P[n][1]);
+            *reinterpret_cast<float2*>(part + 8 * CM_PART + 8 * n) = make_float2(P[n][2], P[n][3]);
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < TASKS; ++k) {
+            const int task = warp + k * WARPS, n = task >> 1, half = task & 1;
+            if (task >= 8) break;
+            const float* src = part_s + (g + 8 * half) * CM_PART + 8 * n + 2 * t;
+            float2 v[WARPS];
+#pragma unroll
+            for (int w = 0; w < WARPS; ++w) v[w] = *reinterpret_cast<const float2*>(src + w * DC_COLS * CM_PART);
+            float2 sum = base[k];
+#pragma unroll
+            for (int w = 0; w < WARPS; w += 2) {
+                sum.x += v[w].x + v[w + 1].x;
+                sum.y += v[w].y + v[w + 1].y;
+            }
+            if (n < 2) {
+                const Pieces x = split3(sum.x, sum.y);
+#pragma unroll
+                for (int p = 0; p < 3; ++p) u_s[(p * 32 + lane) * 4 + 2 * n + half] = x.v[p];
+            } else if (from[k]) {
+                const int r = 8 * (n & 1) + 2 * t, left = total - i * DC_ROWS;
+                float* p = from[k] + i * step[k];
+                if (r < left) p[0] = sum.x;
+                if (r + 1 < left) p[next_row[k]] = sum.y;
+            }
+        }
+        // what does not wait for U: the keys and the decay of the state
+        const uint4* K = M + DP / 16 * CM_M_WORDS / 4;
+        const float* last = reinterpret_cast<const float*>(cm_smem + (i & 1) * BUF + BUF - DP) + 16 * KB * warp + 2 * t;
+        uint32_t b[KB][3][2][2];
+#pragma unroll
+        for (int kb = 0; kb < KB; ++kb) {
+#pragma unroll
+            for (int p = 0; p < 3; ++p) {
+                const uint4 v = K[((warp * KB + kb) * 3 + p) * 32];
+                b[kb][p][0][0] = v.x; b[kb][p][0][1] = v.y; b[kb][p][1][0] = v.z; b[kb][p][1][1] = v.w;
+            }
+#pragma unroll
+            for (int n = 2 * kb; n < 2 * kb + 2; ++n) {
+                const float2 f = *reinterpret_cast<const float2*>(last + 8 * n);
+                S[n][0] *= f.x; S[n][1] *= f.y; S[n][2] *= f.x; S[n][3] *= f.y;
+            }
+        }
+        __syncthreads();
+        uint32_t x[3][4];
+#pragma unroll
+        for (int p = 0; p < 3; ++p) {
+            const uint4 v = *reinterpret_cast<const uint4*>(u_s + (p * 32 + lane) * 4);
+            x[p][0] = v.x; x[p][1] = v.y; x[p][2] = v.z; x[p][3] = v.w;
+        }
+#pragma unroll
+        for (int kb = 0; kb < KB; ++kb) mma_split_pair(S + 2 * kb, x, b[kb]);
+    }
+#pragma unroll
+    for (int n = 0; n < 2 * KB; ++n) {
+        if (in0) *reinterpret_cast<float2*>(own + 8 * n) = make_float2(S[n][0], S[n][1]);
+        if (in1) *reinterpret_cast<float2*>(own + 8 * DP + 8 * n) = make_float2(S[n][2], S[n][3]);
+    }
+}
+
+template <int WARPS, int KB>
+static int launch_carry_mma(const DeltaArgs& a, int n_spans, cudaStream_t stream) {
+    constexpr int smem = carry_mma_words(WARPS, KB) * 4;
+    static bool configured = false;
+    if (!configured) {
+        if (cudaFuncSetAttribute(delta_carry_mma_kernel<WARPS, KB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+            return SHARPI_LAUNCH_FAILED;
+        configured = true;
+    }
+    delta_carry_mma_kernel<WARPS, KB><<<dim3((a.dv + DC_COLS - 1) / DC_COLS, a.heads, n_spans), WARPS * 32, smem, stream>>>(a);
+    SHARPI_CHECK_LAUNCH();
+    return SHARPI_OK;
+}
+
 // `chunks` int32 [n_chunks, 4] (first row, rows <= DC_ROWS, request, unused), a request's one after the other; `spans` int32
-// [n_spans, 4] (request, first chunk, number of chunks, unused); scratch: `mats` [n_chunks * heads * dp * 48], `last`
-// [n_chunks * heads * dp], `u0` [n_chunks * heads * DC_ROWS * dv] floats, each on 16 bytes.
+// [n_spans, 4] (request, first chunk, number of chunks, unused); scratch: `mats` [n_chunks * heads * dp * (split ? 73 : 48)],
+// `last` [n_chunks * heads * dp], `u0` [n_chunks * heads * DC_ROWS * dv] floats, each on 16 bytes.  `split`: the walk over
+// the chunks on the tensor cores (d a multiple of 64).
 SHARPI_API int sharpi_delta_chunks(const float* qkv, const float* beta, const float* z, int ldz, const float* dt_bias,
                                    const float* a_log, const int* row_offsets, const int* state_slots, const int* chunks,
                                    int n_chunks, const int* spans, int n_spans, float* mats, float* last, float* u0,
                                    float* state, long long state_stride, float* y, int kvh, int heads, int d, int dv,
-                                   cudaStream_t stream) {
+                                   int split, cudaStream_t stream) {
     if (n_chunks <= 0) return SHARPI_OK;
     DeltaArgs a;
     if (n_spans <= 0 || n_spans > 65535 || d > DELTA_MAX_CHUNK_KEY ||
@@ -704,18 +964,29 @@ SHARPI_API int sharpi_delta_chunks(const float* qkv, const float* beta, const fl
     const uintptr_t ptrs = reinterpret_cast<uintptr_t>(mats) | reinterpret_cast<uintptr_t>(last);
     if ((ptrs & 15) != 0) return SHARPI_UNALIGNED;
     a.chunks = chunks; a.spans = spans; a.mats = mats; a.last = last; a.u0 = u0;
-    const size_t smem1 = (size_t)3 * DC_ROWS * d * sizeof(float), smem2 = (size_t)delta_carry_floats(a.dp) * sizeof(float);
+    if (split && d % 64 != 0) return SHARPI_BAD_ARGUMENT;
+    const size_t smem1 = ((size_t)3 * DC_ROWS * a.dp + (split ? cm_words(a.dp) : 0)) * sizeof(float), smem2 = (size_t)delta_carry_floats(a.dp) * sizeof(float);
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(delta_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                 (int)(3 * DC_ROWS * DELTA_MAX_CHUNK_KEY * sizeof(float))) != cudaSuccess ||
+        const int most = (int)((3 * DC_ROWS * DELTA_MAX_CHUNK_KEY + cm_words(DELTA_MAX_CHUNK_KEY)) * sizeof(float));
+        if (cudaFuncSetAttribute(delta_chunk_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
+            cudaFuncSetAttribute(delta_chunk_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
             cudaFuncSetAttribute(delta_carry_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)(delta_carry_floats(DELTA_MAX_CHUNK_KEY) * sizeof(float))) != cudaSuccess)
             return SHARPI_LAUNCH_FAILED;
         configured = true;
     }
-    SHARPI_LAUNCH_PDL(delta_chunk_kernel, dim3(n_chunks, heads), DC_THREADS, smem1, stream, a);
-    // the plain way: its blocks run long and are to lie evenly over an empty GPU
+    // the walk over the chunks is launched the plain way: its blocks run long and are to lie evenly over an empty GPU
+    if (split) {
+        SHARPI_LAUNCH_PDL(delta_chunk_kernel<true>, dim3(n_chunks, heads), DC_THREADS, smem1, stream, a);
+        switch (d / 64) {
+            case 1: return launch_carry_mma<4, 1>(a, n_spans, stream);
+            case 2: return launch_carry_mma<8, 1>(a, n_spans, stream);
+            case 3: return launch_carry_mma<6, 2>(a, n_spans, stream);
+            default: return launch_carry_mma<8, 2>(a, n_spans, stream);
+        }
+    }
+    SHARPI_LAUNCH_PDL(delta_chunk_kernel<false>, dim3(n_chunks, heads), DC_THREADS, smem1, stream, a);
     delta_carry_kernel<<<dim3((dv + DC_COLS - 1) / DC_COLS, heads, n_spans), DC_THREADS, smem2, stream>>>(a);
     SHARPI_CHECK_LAUNCH();
     return SHARPI_OK;

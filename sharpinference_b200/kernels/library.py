@@ -100,7 +100,7 @@ SIGNATURES: Dict[str, Tuple[str, list]] = {
     "sharpi_side_gate": ("sandwich", [P, I, P, P, I, LL, I, I, I, P, I, I, I, P]),
     "sharpi_delta_prep": ("delta", [P, I, P, P, LL, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P]),
     "sharpi_delta_walk": ("delta", [P, P, P, I, P, P, P, P, P, I, I, P, LL, P, I, I, I, I, P]),
-    "sharpi_delta_chunks": ("delta", [P, P, P, I, P, P, P, P, P, I, P, I, P, P, P, P, LL, P, I, I, I, I, P]),
+    "sharpi_delta_chunks": ("delta", [P, P, P, I, P, P, P, P, P, I, P, I, P, P, P, P, LL, P, I, I, I, I, I, P]),
     "sharpi_head_norm_gate": ("delta", [P, P, I, P, F, I, I, I, P, I, P]),
     "sharpi_gated_group_norm": ("mamba2", [P, P, I, P, F, I, I, I, P, I, P]),
 }

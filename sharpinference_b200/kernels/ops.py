@@ -1888,12 +1888,15 @@ def delta_prep(proj: torch.Tensor, *, conv_weight: torch.Tensor, conv_state: Opt
 def delta_rule(qkv: torch.Tensor, beta: torch.Tensor, z: torch.Tensor, *, dt_bias: torch.Tensor, a_log: torch.Tensor,
                row_offsets: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, kv_heads: int, heads: int, d: int,
                dv: int, num_requests: int, walk_requests: Optional[torch.Tensor] = None, num_walk: Optional[int] = None,
-               chunks: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None, max_rows: int = 1) -> torch.Tensor:
+               chunks: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None, max_rows: int = 1,
+               split: bool = False) -> torch.Tensor:
     """``S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q`` per head, ``g = exp(-exp(a_log) softplus(z + dt_bias))`` per
     key channel: float32 ``[T, heads * dv]``.  ``qkv`` and ``beta`` as :func:`delta_prep` leaves them, ``z`` float32
     ``[T, heads * d]`` (possibly a column range), ``state`` ``[slots, delta_state_floats]``.  ``walk_requests`` (None: all) are
     walked row by row, the requests of ``spans`` (int32 ``[m, 4]``) by chunks (int32 ``[n, 4]``, at most DELTA_CHUNK rows).
-    ``max_rows``: the most rows a walked request brings (it decides how the kernel is launched and changes no result)."""
+    ``max_rows``: the most rows a walked request brings (it decides how the kernel is launched and changes no result).  ``split``:
+    where the key size is a multiple of 64, the chunks' products run on the tensor cores with every operand cut into bfloat16
+    pieces of 24 bits together."""
     ldz = _need_columns(z, "z", torch.float32)
     for name, t in (("qkv", qkv), ("beta", beta), ("dt_bias", dt_bias), ("a_log", a_log), ("state", state)):
         _need(t, name, torch.float32)
@@ -1913,12 +1916,13 @@ def delta_rule(qkv: torch.Tensor, beta: torch.Tensor, z: torch.Tensor, *, dt_bia
         _need(chunks, "chunks", torch.int32)
         _need(spans, "spans", torch.int32)
         n, dp = chunks.shape[0], (d + 3) // 4 * 4
-        mats = torch.empty((n * heads * dp, 3 * DELTA_CHUNK), dtype=torch.float32, device=qkv.device)
+        split = split and d % 64 == 0
+        mats = torch.empty((n * heads * dp, 73 if split else 3 * DELTA_CHUNK), dtype=torch.float32, device=qkv.device)
         last = torch.empty((n * heads, dp), dtype=torch.float32, device=qkv.device)
         u0 = torch.empty((n * heads * DELTA_CHUNK, dv), dtype=torch.float32, device=qkv.device)
         check(kernel("sharpi_delta_chunks")(*common, chunks.data_ptr(), n, spans.data_ptr(), spans.shape[0], mats.data_ptr(),
                                             last.data_ptr(), u0.data_ptr(), state.data_ptr(), state.stride(0), y.data_ptr(),
-                                            kv_heads, heads, d, dv, _stream()), "sharpi_delta_chunks")
+                                            kv_heads, heads, d, dv, int(split), _stream()), "sharpi_delta_chunks")
     if n_walk:
         if walk_requests is not None:
             _need(walk_requests, "walk_requests", torch.int32)

@@ -10,7 +10,8 @@ with ``conv`` a short causal convolution per channel.  The fused projection's co
 low-rank maps go on through one product whose weight holds ``W2`` and ``G2`` on its diagonal (the low-rank columns are padded
 to a multiple of 8).  Per-request state, float32: ``S`` (``state_specs["S"]``, a column of ``d`` numbers per value element) and
 the convolutions' last ``taps - 1`` inputs (``state_specs["conv"]``).  Convolutions, unit norms, steps, decays, the state, all
-its sums and the norm are float32 (``csrc/delta.cu``).  A request that brings few rows is walked row by row; longer portions
+its sums and the norm are float32 (``csrc/delta.cu``; a bfloat16 model's long portions form the products with the state on the
+tensor cores, every operand in bfloat16 pieces of 24 bits together).  A request that brings few rows is walked row by row; longer portions
 are cut into chunks (:class:`DeltaPlanner`).
 """
 from __future__ import annotations
@@ -37,7 +38,7 @@ class DeltaPlanner(StepPlanner):
     rows, request, 0), a request's one after the other, and ``spans`` ``[m, 4]`` (request, first chunk, chunks, 0).  Which of
     the two a request is depends on its own rows alone.  A tile has at least as many rows as a convolution looks back."""
 
-    WALK_ROWS_UP_TO = 32
+    WALK_ROWS_UP_TO = 24        # (16 heads of 128 x 128: 16 rows 14 us walked, 19 us in chunks; 32 rows 23 and 20 us)
     TILE_ROWS = 8
 
     def __init__(self, taps: int, chunked: bool):
@@ -117,5 +118,5 @@ class ChannelDelta(Mixer):
         y = ops.delta_rule(qkv, beta, z[:, :n], dt_bias=self.dt_bias, a_log=self.a_log, row_offsets=ctx.row_offsets,
                            state_slots=ctx.state_slots, state=slot.states["S"], num_requests=ctx.num_requests,
                            walk_requests=plan.walk, num_walk=plan.num_walk, chunks=plan.chunks, spans=plan.spans,
-                           max_rows=plan.walk_rows, **sizes)
+                           max_rows=plan.walk_rows, split=self.act_dtype == torch.bfloat16, **sizes)
         return self.out(ops.head_norm_gate(y, z[:, n:], self.norm_weight, self.eps, self.heads, self.act_dtype))

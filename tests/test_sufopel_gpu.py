@@ -266,9 +266,11 @@ def _delta_case(n, G, H, d, dv, seed, kind):
 
 
 @pytest.mark.parametrize("kind", ["mixed", "slow", "strong"])
-@pytest.mark.parametrize("G,H,d,dv", [(2, 2, 32, 32), (1, 3, 5, 7), (1, 1, 128, 128), (2, 4, 64, 40), (1, 1, 160, 72), (1, 2, 300, 24),
-                                      (1, 2, 1, 1), (1, 1, 96, 200), (1, 2, 256, 16), (1, 1, 36, 17)])
-def test_delta_rule_walked_and_in_chunks(G, H, d, dv, kind):
+@pytest.mark.parametrize("G,H,d,dv,split", [(2, 2, 32, 32, False), (1, 3, 5, 7, False), (1, 2, 192, 33, False), (1, 2, 192, 33, True),
+                                            (1, 1, 128, 128, False), (1, 1, 128, 128, True), (2, 4, 64, 40, False), (2, 4, 64, 40, True),
+                                            (1, 1, 160, 72, False), (1, 2, 300, 24, False), (1, 2, 1, 1, False), (1, 1, 96, 200, False),
+                                            (1, 2, 256, 16, False), (1, 2, 256, 17, True), (1, 1, 36, 17, False)])
+def test_delta_rule_walked_and_in_chunks(G, H, d, dv, split, kind):
     """Three requests on slots of their own, in portions of one to 150 rows, walked and in chunks of 16 (also a last chunk of one
     row), against the rows one by one; the two forms continue one another's state.  Decays near 1 throughout, spread, and ones
     that are zero in 32-bit: a closed form that divides by a product of decays, or sums their logarithms, fails on the last."""
@@ -293,7 +295,7 @@ def test_delta_rule_walked_and_in_chunks(G, H, d, dv, kind):
         off = [0, lens[0], lens[0] + lens[1], sum(lens)]
         y = ops.delta_rule(f32(qkv), f32(cut(3, 0)), f32(z)[:, 3: 3 + H * d], dt_bias=f32(bias), a_log=f32(a_log), row_offsets=i32(off),
                            state_slots=i32(slots), state=state, kv_heads=G, heads=H, d=d, dv=dv, num_requests=3, walk_requests=dev["walk"],
-                           num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"], max_rows=plan.values["walk_rows"]).cpu()
+                           num_walk=plan.values["num_walk"], chunks=dev["chunks"], spans=dev["spans"], max_rows=plan.values["walk_rows"], split=split).cpu()
         for b in range(3):
             got[b].append(y[off[b]: off[b + 1]])
             at[b] += lens[b]
