@@ -27,6 +27,8 @@
 // Norm sums, angles, sines and cosines are float32; a row's numbers depend on the row alone.
 #include "common.cuh"
 
+#include <initializer_list>
+
 constexpr int LAT_THREADS = 128;
 
 template <typename TO>
@@ -103,17 +105,54 @@ SHARPI_API int sharpi_latent_down_post(const float* down, int ld, int q_rank, in
     return SHARPI_OK;
 }
 
-template <typename TS, typename TO>
+// Four neighbouring elements a thread where sizes, strides and addresses allow it.
+template <int VEC> __device__ __forceinline__ void load_vec(const float* p, float* v) {
+    if (VEC == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        v[0] = x.x; v[1 % VEC] = x.y; v[2 % VEC] = x.z; v[3 % VEC] = x.w;
+    } else {
+        v[0] = *p;
+    }
+}
+template <int VEC> __device__ __forceinline__ void load_vec(const bf16* p, float* v) {
+    if (VEC == 4) {
+        const uint2 x = *reinterpret_cast<const uint2*>(p);
+        v[0] = __uint_as_float(x.x << 16); v[1 % VEC] = __uint_as_float(x.x & 0xffff0000u);
+        v[2 % VEC] = __uint_as_float(x.y << 16); v[3 % VEC] = __uint_as_float(x.y & 0xffff0000u);
+    } else {
+        v[0] = to_float(*p);
+    }
+}
+template <int VEC> __device__ __forceinline__ void store_vec(float* p, const float* v) {
+    if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]);
+    else *p = v[0];
+}
+template <int VEC> __device__ __forceinline__ void store_vec(bf16* p, const float* v) {
+    if (VEC == 4) {
+        __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1 % VEC]), b = __floats2bfloat162_rn(v[2 % VEC], v[3 % VEC]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&a), *reinterpret_cast<unsigned*>(&b));
+    } else {
+        *p = from_float<bf16>(v[0]);
+    }
+}
+static inline bool fours(std::initializer_list<long long> sizes, std::initializer_list<const void*> pointers) {
+    for (long long n : sizes)
+        if (n % 4 != 0) return false;
+    for (const void* p : pointers)
+        if (reinterpret_cast<uintptr_t>(p) & 15) return false;
+    return true;
+}
+
+template <typename TS, typename TO, int VEC>
 __global__ void __launch_bounds__(256)
 head_major_kernel(const TS* src, int T, int heads, int stride, int col0, int n, TO* dst, int ld) {
     pdl_wait();
-    const long long total = (long long)T * heads * n;
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= total) return;
-    const int c = (int)(i % n);
-    const long long th = i / n;
-    const int t = (int)(th % T), h = (int)(th / T);
-    dst[i] = from_float<TO>(to_float(src[(size_t)t * ld + (size_t)h * stride + col0 + c]));
+    const int t = blockIdx.x, i = blockIdx.y * blockDim.x + threadIdx.x, per = n / VEC;
+    const int h = i / per, c = i % per * VEC;
+    if (h >= heads) return;
+    float v[VEC];
+    load_vec<VEC>(src + (size_t)t * ld + (size_t)h * stride + col0 + c, v);
+    store_vec<VEC>(dst + ((size_t)h * T + t) * n + c, v);
 }
 
 SHARPI_API int sharpi_head_major(const void* src, int src_dtype, int T, int heads, int stride, int col0, int n,
@@ -121,77 +160,94 @@ SHARPI_API int sharpi_head_major(const void* src, int src_dtype, int T, int head
     if (T <= 0 || n <= 0) return SHARPI_OK;
     if (ld <= 0) ld = heads * stride;          // rows lie end to end
     if (heads <= 0 || col0 < 0 || col0 + n > stride || ld < heads * stride) return SHARPI_BAD_ARGUMENT;
-    const long long total = (long long)T * heads * n;
-    const unsigned blocks = (unsigned)((total + 255) / 256);
-    if (src_dtype == SHARPI_F32 && dst_dtype == SHARPI_F32)
-        SHARPI_LAUNCH_PDL((head_major_kernel<float, float>), blocks, 256, 0, stream, (const float*)src, T, heads, stride, col0, n, (float*)dst, ld);
-    else if (src_dtype == SHARPI_F32 && dst_dtype == SHARPI_BF16)
-        SHARPI_LAUNCH_PDL((head_major_kernel<float, bf16>), blocks, 256, 0, stream, (const float*)src, T, heads, stride, col0, n, (bf16*)dst, ld);
-    else if (src_dtype == SHARPI_BF16 && dst_dtype == SHARPI_BF16)
-        SHARPI_LAUNCH_PDL((head_major_kernel<bf16, bf16>), blocks, 256, 0, stream, (const bf16*)src, T, heads, stride, col0, n, (bf16*)dst, ld);
+    const bool vec = fours({n, stride, col0, ld}, {src, dst});
+    const dim3 grid(T, ((long long)heads * (n / (vec ? 4 : 1)) + 255) / 256);
+#define MAJOR_CASE(TS, TO)                                                                                                       \
+    do {                                                                                                                         \
+        if (vec) SHARPI_LAUNCH_PDL((head_major_kernel<TS, TO, 4>), grid, 256, 0, stream, (const TS*)src, T, heads, stride, col0, n, (TO*)dst, ld); \
+        else SHARPI_LAUNCH_PDL((head_major_kernel<TS, TO, 1>), grid, 256, 0, stream, (const TS*)src, T, heads, stride, col0, n, (TO*)dst, ld); \
+    } while (0)
+    if (src_dtype == SHARPI_F32 && dst_dtype == SHARPI_F32) MAJOR_CASE(float, float);
+    else if (src_dtype == SHARPI_F32 && dst_dtype == SHARPI_BF16) MAJOR_CASE(float, bf16);
+    else if (src_dtype == SHARPI_BF16 && dst_dtype == SHARPI_BF16) MAJOR_CASE(bf16, bf16);
     else
         return SHARPI_BAD_ARGUMENT;
+#undef MAJOR_CASE
     return SHARPI_OK;
 }
 
-template <typename TO>
+template <typename TO, int VEC>
 __global__ void __launch_bounds__(256)
 head_minor_kernel(const float* src, int T, int heads, int stride, int col0, int n, TO* dst, const float* gate,
                   int gate_ld, int gate_elem) {
     pdl_wait();
-    const long long total = (long long)T * heads * n;
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= total) return;
-    const int c = (int)(i % n);
-    const long long th = i / n;
-    const int h = (int)(th % heads), t = (int)(th / heads);
-    float v = src[((size_t)h * T + t) * n + c];
-    if (gate) v = v / (1.0f + expf(-gate[(size_t)t * gate_ld + (gate_elem ? h * n + c : h)]));      // times sigmoid(gate logit)
-    dst[((size_t)t * heads + h) * stride + col0 + c] = from_float<TO>(v);
+    const int t = blockIdx.x, i = blockIdx.y * blockDim.x + threadIdx.x, per = n / VEC;
+    const int h = i / per, c = i % per * VEC;
+    if (h >= heads) return;
+    float v[VEC], z[VEC];
+    load_vec<VEC>(src + ((size_t)h * T + t) * n + c, v);
+    if (gate) {                                                        // times sigmoid(gate logit)
+        if (gate_elem) {
+            load_vec<VEC>(gate + (size_t)t * gate_ld + h * n + c, z);
+#pragma unroll
+            for (int u = 0; u < VEC; ++u) v[u] = v[u] / (1.0f + expf(-z[u]));
+        } else {
+            const float e = expf(-gate[(size_t)t * gate_ld + h]);
+#pragma unroll
+            for (int u = 0; u < VEC; ++u) v[u] = v[u] / (1.0f + e);
+        }
+    }
+    store_vec<VEC>(dst + ((size_t)t * heads + h) * stride + col0 + c, v);
 }
 
 SHARPI_API int sharpi_head_minor(const float* src, int T, int heads, int stride, int col0, int n, void* dst,
                                  int dst_dtype, const float* gate, int gate_ld, int gate_elem, cudaStream_t stream) {
     if (T <= 0 || n <= 0) return SHARPI_OK;
     if (heads <= 0 || col0 < 0 || col0 + n > stride) return SHARPI_BAD_ARGUMENT;
-    const long long total = (long long)T * heads * n;
-    const unsigned blocks = (unsigned)((total + 255) / 256);
-    if (dst_dtype == SHARPI_F32)
-        SHARPI_LAUNCH_PDL(head_minor_kernel<float>, blocks, 256, 0, stream, src, T, heads, stride, col0, n, (float*)dst, gate, gate_ld, gate_elem);
-    else if (dst_dtype == SHARPI_BF16)
-        SHARPI_LAUNCH_PDL(head_minor_kernel<bf16>, blocks, 256, 0, stream, src, T, heads, stride, col0, n, (bf16*)dst, gate, gate_ld, gate_elem);
+    const bool vec = fours({n, stride, col0, gate && gate_elem ? gate_ld : 0}, {src, dst, gate && gate_elem ? gate : nullptr});
+    const dim3 grid(T, ((long long)heads * (n / (vec ? 4 : 1)) + 255) / 256);
+#define MINOR_CASE(TO)                                                                                                           \
+    do {                                                                                                                         \
+        if (vec) SHARPI_LAUNCH_PDL((head_minor_kernel<TO, 4>), grid, 256, 0, stream, src, T, heads, stride, col0, n, (TO*)dst, gate, gate_ld, gate_elem); \
+        else SHARPI_LAUNCH_PDL((head_minor_kernel<TO, 1>), grid, 256, 0, stream, src, T, heads, stride, col0, n, (TO*)dst, gate, gate_ld, gate_elem); \
+    } while (0)
+    if (dst_dtype == SHARPI_F32) MINOR_CASE(float);
+    else if (dst_dtype == SHARPI_BF16) MINOR_CASE(bf16);
     else
         return SHARPI_BAD_ARGUMENT;
+#undef MINOR_CASE
     return SHARPI_OK;
 }
 
-template <typename TO>
+template <typename TO, int VEC>                        // VEC 4: rank, rot and D are multiples of 4
 __global__ void __launch_bounds__(256)
 latent_q_join_kernel(const float* qa, const float* q, const int* positions, const float* __restrict__ inv_freq, int T,
                      int heads, int dim, int rank, int rot, int rot_dims, int D, TO* dst, int ldq, float rot_amp) {
     pdl_wait();
-    const long long total = (long long)T * heads * D;
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= total) return;
-    const int c = (int)(i % D);
-    const long long th = i / D;
-    const int h = (int)(th % heads), t = (int)(th / heads);
-    float v = 0.0f;
-    if (c < rank) {
-        v = qa[((size_t)h * T + t) * rank + c];
-    } else if (c < rank + rot) {
-        const int j = c - rank;
-        const float* qr = q + (size_t)t * ldq + (size_t)h * (dim + rot) + dim;
-        v = qr[j];
-        if (j < rot_dims && inv_freq) {
-            float sn, cs;
-            sincosf((float)positions[t] * inv_freq[j >> 1], &sn, &cs);
-            sn *= rot_amp;
-            cs *= rot_amp;
-            v = (j & 1) ? qr[j] * cs + qr[j - 1] * sn : qr[j] * cs - qr[j + 1] * sn;
+    const int t = blockIdx.x, i = blockIdx.y * blockDim.x + threadIdx.x, per = D / VEC;
+    const int h = i / per, c0 = i % per * VEC;
+    if (h >= heads) return;
+    float v[VEC];
+    if (c0 + VEC <= rank) {
+        load_vec<VEC>(qa + ((size_t)h * T + t) * rank + c0, v);
+    } else {
+#pragma unroll
+        for (int u = 0; u < VEC; ++u) {
+            const int j = c0 + u - rank;
+            v[u] = 0.0f;
+            if (j < 0 || j >= rot) continue;
+            const float* qr = q + (size_t)t * ldq + (size_t)h * (dim + rot) + dim;
+            v[u] = qr[j];
+            if (j < rot_dims && inv_freq) {
+                float sn, cs;
+                sincosf((float)positions[t] * inv_freq[j >> 1], &sn, &cs);
+                sn *= rot_amp;
+                cs *= rot_amp;
+                v[u] = (j & 1) ? qr[j] * cs + qr[j - 1] * sn : qr[j] * cs - qr[j + 1] * sn;
+            }
         }
     }
-    dst[i] = from_float<TO>(v);
+    store_vec<VEC>(dst + ((size_t)t * heads + h) * D + c0, v);
 }
 
 SHARPI_API int sharpi_latent_q_join(const float* qa, const float* q, const int* positions, const float* inv_freq,
@@ -202,15 +258,17 @@ SHARPI_API int sharpi_latent_q_join(const float* qa, const float* q, const int* 
     if (heads <= 0 || dim <= 0 || rank <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || (rot_dims & 1) ||
         rank + rot > D)
         return SHARPI_BAD_ARGUMENT;
-    const long long total = (long long)T * heads * D;
-    const unsigned blocks = (unsigned)((total + 255) / 256);
-    if (dst_dtype == SHARPI_F32)
-        SHARPI_LAUNCH_PDL(latent_q_join_kernel<float>, blocks, 256, 0, stream, qa, q, positions, inv_freq, T, heads,
-                          dim, rank, rot, rot_dims, D, (float*)dst, ldq, rot_amp);
-    else if (dst_dtype == SHARPI_BF16)
-        SHARPI_LAUNCH_PDL(latent_q_join_kernel<bf16>, blocks, 256, 0, stream, qa, q, positions, inv_freq, T, heads,
-                          dim, rank, rot, rot_dims, D, (bf16*)dst, ldq, rot_amp);
+    const bool vec = fours({rank, rot, D}, {qa, dst});
+    const dim3 grid(T, ((long long)heads * (D / (vec ? 4 : 1)) + 255) / 256);
+#define JOIN_CASE(TO)                                                                                                            \
+    do {                                                                                                                         \
+        if (vec) SHARPI_LAUNCH_PDL((latent_q_join_kernel<TO, 4>), grid, 256, 0, stream, qa, q, positions, inv_freq, T, heads, dim, rank, rot, rot_dims, D, (TO*)dst, ldq, rot_amp); \
+        else SHARPI_LAUNCH_PDL((latent_q_join_kernel<TO, 1>), grid, 256, 0, stream, qa, q, positions, inv_freq, T, heads, dim, rank, rot, rot_dims, D, (TO*)dst, ldq, rot_amp); \
+    } while (0)
+    if (dst_dtype == SHARPI_F32) JOIN_CASE(float);
+    else if (dst_dtype == SHARPI_BF16) JOIN_CASE(bf16);
     else
         return SHARPI_BAD_ARGUMENT;
+#undef JOIN_CASE
     return SHARPI_OK;
 }

@@ -216,31 +216,49 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-template <typename TT, typename TO>
+template <typename TT, typename TO, int VEC>                    // VEC neighbouring columns a thread
 __global__ void __launch_bounds__(128)
 side_gate_kernel(const float* gate, int ld, const int* ids, const TT* __restrict__ table, long long ld_table, int col0, int n,
-                 int n_out, TO* out, int T, int V) {
+                 int n_out, TO* out, unsigned total, int V) {
     pdl_wait();
-    const long long total = (long long)T * n_out;
-    const long long i = (long long)blockIdx.x * 128 + threadIdx.x;
+    const unsigned i = blockIdx.x * 128 + threadIdx.x;
     if (i >= total) return;
-    const int t = (int)(i / n_out), j = (int)(i % n_out);
-    float v = 0.0f;
-    if (j < n) {
-        const int id = ids[t];
-        if (id >= 0 && id < V) v = gelu_tanh_f(gate[(size_t)t * ld + j]) * to_float(table[(size_t)id * ld_table + col0 + j]);
+    const unsigned per = n_out / VEC;
+    const int t = (int)(i / per), j = (int)(i % per) * VEC;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < V;
+    const TT* e = table + (size_t)(ok ? id : 0) * ld_table + col0 + j;
+    const float* z = gate + (size_t)t * ld + j;
+    float g[VEC], v[VEC];
+#pragma unroll
+    for (int u = 0; u < VEC; ++u) g[u] = j + u < n ? z[u] : 0.0f;
+#pragma unroll
+    for (int u = 0; u < VEC; ++u) v[u] = ok && j + u < n ? to_float(e[u]) : 0.0f;
+#pragma unroll
+    for (int u = 0; u < VEC; ++u) v[u] *= gelu_tanh_f(g[u]);
+    if (VEC == 4) {
+        store4<TO>(out + (size_t)t * n_out + j, v);
+    } else {
+        out[(size_t)t * n_out + j] = from_float<TO>(v[0]);
     }
-    out[i] = from_float<TO>(v);
 }
 
 SHARPI_API int sharpi_side_gate(const float* gate, int ld, const int* ids, const void* table, int table_dtype, long long ld_table,
                                 int col0, int n, int n_out, void* out, int out_dtype, int T, int V, cudaStream_t stream) {
     if (T <= 0) return SHARPI_OK;
     if (n <= 0 || n_out < n || col0 < 0 || col0 + n > ld_table || ld < n || V <= 0) return SHARPI_BAD_ARGUMENT;
-    const unsigned blocks = (unsigned)(((long long)T * n_out + 127) / 128);
-#define SIDE_CASE(TT, TO)                                                                                                    \
-    SHARPI_LAUNCH_PDL((side_gate_kernel<TT, TO>), blocks, 128, 0, stream, gate, ld, ids, (const TT*)table, ld_table, col0, n, \
-                      n_out, (TO*)out, T, V)
+    const int vec = n_out % 4 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 ? 4 : 1;
+    if ((long long)T * n_out > 0x7fffffffLL) return SHARPI_BAD_ARGUMENT;
+    const unsigned total = (unsigned)T * (unsigned)(n_out / vec), blocks = (total + 127) / 128;
+#define SIDE_CASE(TT, TO)                                                                                                      \
+    do {                                                                                                                       \
+        if (vec == 4)                                                                                                          \
+            SHARPI_LAUNCH_PDL((side_gate_kernel<TT, TO, 4>), blocks, 128, 0, stream, gate, ld, ids, (const TT*)table, ld_table, \
+                              col0, n, n_out, (TO*)out, total, V);                                                             \
+        else                                                                                                                   \
+            SHARPI_LAUNCH_PDL((side_gate_kernel<TT, TO, 1>), blocks, 128, 0, stream, gate, ld, ids, (const TT*)table, ld_table, \
+                              col0, n, n_out, (TO*)out, total, V);                                                             \
+    } while (0)
     if (table_dtype == SHARPI_F32 && out_dtype == SHARPI_F32) SIDE_CASE(float, float);
     else if (table_dtype == SHARPI_BF16 && out_dtype == SHARPI_BF16) SIDE_CASE(bf16, bf16);
     else if (table_dtype == SHARPI_F32 && out_dtype == SHARPI_BF16) SIDE_CASE(float, bf16);
